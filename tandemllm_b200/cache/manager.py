@@ -128,6 +128,8 @@ class CacheManager:
             if isinstance(need, PagedNeed):
                 if need.window is not None and need.window <= 0:
                     raise ValueError(f"site {i}: window {need.window} must be positive")
+                if need.chunk is not None and (need.chunk <= 0 or need.window is not None):
+                    raise ValueError(f"site {i}: chunks of {need.chunk} positions: a positive size, and no window beside it")
                 if need not in by_need:
                     by_need[need] = PageGroup(need, [], PagePool(num_pages), page_size)
                     self.groups.append(by_need[need])
@@ -224,14 +226,14 @@ class CacheManager:
                 g.extend(req, g.pool.take(need, req))
 
     def advance(self, req, new_len: int) -> None:
-        """The request now holds `new_len` tokens: windowed groups give back the pages no later row can read."""
+        """The request now holds `new_len` tokens: windowed and chunked groups give back the pages no later row can read."""
         self._length[req] = new_len
         for g in self.groups:
-            w = g.need.window
-            if w is None:
+            w, chunk = g.need.window, g.need.chunk
+            if w is None and chunk is None:
                 continue
-            # the next row sits at position new_len and reads positions >= new_len - w + 1
-            first_needed = max(0, new_len - w + 1) // g.page_size
+            # the next row sits at position new_len and reads positions >= new_len - w + 1, or its own chunk's
+            first_needed = (max(0, new_len - w + 1) if w is not None else new_len - new_len % chunk) // g.page_size
             kept = -(-g.need.keep_first // g.page_size)       # pages that hold positions every later row still reads
             table = g.tables[req]
             stop = min(first_needed, len(table))
@@ -269,7 +271,7 @@ class CacheManager:
             "page_size": self.page_size,
             "requests": len(self._slot_of),
             "free_slots": len(self._free_slots),
-            "groups": [{"sites": len(g.sites), "window": g.need.window, "pages": g.pool.num_pages, "free": g.pool.free,
+            "groups": [{"sites": len(g.sites), "window": g.need.window, "chunk": g.need.chunk, "pages": g.pool.num_pages, "free": g.pool.free,
                         "peak_used": g.pool.peak_used, "reused": g.pool.reused} for g in self.groups],
         }
 

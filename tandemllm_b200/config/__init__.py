@@ -1,5 +1,8 @@
 """Configuration: the typed per-architecture readers, the neutral `ModelSpec`, and the registry."""
 
+from .gifopel import ARCHITECTURES as _GIFOPEL_ARCHS
+from .gifopel import MODEL_TYPES as _GIFOPEL_TYPES
+from .gifopel import GifopelConfig
 from .lfm2_moe import ARCHITECTURES as _LFM2_ARCHS
 from .lfm2_moe import MODEL_TYPES as _LFM2_TYPES
 from .lfm2_moe import Lfm2MoeConfig
@@ -34,6 +37,9 @@ register(Architecture(name="sebilorn", architectures=_SEBILORN_ARCHS, model_type
 register(Architecture(name="niralix", architectures=_NIRALIX_ARCHS, model_types=_NIRALIX_TYPES,
                       read_config=NiralixConfig.from_dict))
 
-__all__ = ["NiralixConfig", "PuripelConfig", "SebilornConfig", "REGISTRY", "Architecture", "architecture_of", "read_model_config", "register", "unregister",
+register(Architecture(name="gifopel", architectures=_GIFOPEL_ARCHS, model_types=_GIFOPEL_TYPES,
+                      read_config=GifopelConfig.from_dict))
+
+__all__ = ["GifopelConfig", "NiralixConfig", "PuripelConfig", "SebilornConfig", "REGISTRY", "Architecture", "architecture_of", "read_model_config", "register", "unregister",
            "resolve_model_folder", "spec_of", "LayerSpec", "ModelSpec", "PartSpec", "Site", "StreamAdd", "plain_schedule",
            "Lfm2MoeConfig", "SifupelConfig"]

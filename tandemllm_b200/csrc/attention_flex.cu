@@ -1,16 +1,19 @@
 // Attention over the paged cache with the options a design may combine, on the CUDA cores, in 32-bit or bfloat16 storage
 // with 32-bit arithmetic; any head size up to 256 for keys and, separately, for values.
 //
-//   tl_qkv_rotate_store   one row a block: q, k (first `rot` entries of a head turned by the row's position, halves
-//                         layout: entry i with entry i + rot / 2) and v (optionally turned over all its entries with
+//   tl_qkv_rotate_store   one row a block: q, k (first `rot` entries of a head turned by the row's position, in the halves
+//                         layout, entry i with entry i + rot / 2, or the interleaved one, entry 2i with entry 2i + 1; before
+//                         that optionally divided by the head's root mean square, times a weight the heads share) and v (optionally turned over all its entries with
 //                         frequencies of its own) from one fused product; q to a plain tensor, k and v into their pages.
 //                         The sines and cosines of q and k may carry a common factor (a stretched rotation's magnitude);
 //                         v may first be blended with another tensor's values of the same row, (1 - l) v + l v_other, l a
 //                         number on the device (values carried over from an earlier layer)
 //   tl_attention_flex     one warp a (row, query head): score = scale q.k, optionally capped (c tanh(score / c)); row at
-//                         position i sees key j <= i when there is no window, or i - j < window, or j < keep_first;
-//                         softmax in 32-bit; the output optionally turned back by the row's own position (the inverse of
-//                         the values' turn), optionally times sigmoid(gate) entry by entry, times `out_scale`
+//                         position i sees key j <= i when there is no window, or i - j < window, or j < keep_first, or, with
+//                         chunks, when i and j lie in the same chunk of positions; softmax in 32-bit, its denominator
+//                         optionally with exp(sink) of a number a head (no key, no value); the output optionally turned back by the row's own position (the inverse of
+//                         the values' turn), optionally times sigmoid(gate) entry by entry or head by head, times
+//                         `out_scale`
 //
 // Cache layout per site: K [pages, kv heads, page_size, D], V [pages, kv heads, page_size, VD]. Keys are visited in
 // chunks of 32 aligned to absolute positions (first the kept first tokens that lie before the window, then the window)
@@ -22,12 +25,16 @@ namespace tl {
 
 constexpr int FLEX_MAX_DIM = 256;
 
+// Entry i of a head x, times inv and its weight where the head is normed (w null: as it is), then turned with its partner.
 template <typename T>
 __device__ __forceinline__ float rotated_entry(const T* __restrict__ x, int i, int half, const float* __restrict__ sn,
-                                               const float* __restrict__ cs) {
-  if (i < half) return to_f32(x[i]) * cs[i] - to_f32(x[i + half]) * sn[i];
-  if (i < 2 * half) return to_f32(x[i]) * cs[i - half] + to_f32(x[i - half]) * sn[i - half];
-  return to_f32(x[i]);
+                                               const float* __restrict__ cs, const float* __restrict__ w = nullptr, float inv = 1.f,
+                                               bool neighbours = false) {
+  auto at = [&](int e) { return w ? to_f32(x[e]) * inv * w[e] : to_f32(x[e]); };
+  if (i >= 2 * half) return at(i);
+  if (neighbours) return (i & 1) ? at(i) * cs[i >> 1] + at(i - 1) * sn[i >> 1] : at(i) * cs[i >> 1] - at(i + 1) * sn[i >> 1];
+  if (i < half) return at(i) * cs[i] - at(i + half) * sn[i];
+  return at(i) * cs[i - half] + at(i - half) * sn[i - half];
 }
 
 template <typename T>
@@ -36,7 +43,9 @@ __global__ void __launch_bounds__(128) qkv_rotate_store_kernel(
     const float* __restrict__ inv_freq_v, const int* __restrict__ positions, const int* __restrict__ req_of_row,
     const int* __restrict__ block_table, int max_pages, int page_size, int num_pages, T* __restrict__ q_out,
     T* __restrict__ k_cache, T* __restrict__ v_cache, int Hq, int Hk, int D, int VD, int* __restrict__ status,
-    float rot_magnitude, const T* __restrict__ v_other, long long ld_other, const float* __restrict__ v_blend) {
+    float rot_magnitude, const T* __restrict__ v_other, long long ld_other, const float* __restrict__ v_blend,
+    const float* __restrict__ q_weight, const float* __restrict__ k_weight, float norm_eps, int neighbours) {
+  extern __shared__ float head_inv[];           // [Hq + Hk] with q/k norms: 1 / rms of every head
   __shared__ float sn[FLEX_MAX_DIM / 2], cs[FLEX_MAX_DIM / 2], snv[FLEX_MAX_DIM / 2], csv[FLEX_MAX_DIM / 2];
   const int r = blockIdx.x;
   const int pos = positions[r];
@@ -47,11 +56,25 @@ __global__ void __launch_bounds__(128) qkv_rotate_store_kernel(
     cs[i] *= rot_magnitude;
   }
   for (int i = threadIdx.x; i < vhalf; i += blockDim.x) sincosf((float)pos * inv_freq_v[i], &snv[i], &csv[i]);
-  __syncthreads();
   const T* row = qkv + (long long)r * ld;
+  if (q_weight) {
+    const int lane = threadIdx.x & 31;
+    for (int h = threadIdx.x >> 5; h < Hq + (k_col >= 0 ? Hk : 0); h += blockDim.x >> 5) {
+      const T* x = row + (h < Hq ? q_col + h * D : k_col + (h - Hq) * D);
+      float ss = 0.f;
+      for (int i = lane; i < D; i += 32) {
+        const float v = to_f32(x[i]);
+        ss = fmaf(v, v, ss);
+      }
+      ss = warp_sum(ss);
+      if (lane == 0) head_inv[h] = 1.f / sqrtf(ss / (float)D + norm_eps);
+    }
+  }
+  __syncthreads();
   for (int e = threadIdx.x; e < Hq * D; e += blockDim.x) {
     const int h = e / D, i = e - h * D;
-    q_out[(long long)r * Hq * D + e] = from_f32<T>(rotated_entry(row + q_col + h * D, i, half, sn, cs));
+    q_out[(long long)r * Hq * D + e] = from_f32<T>(rotated_entry(row + q_col + h * D, i, half, sn, cs, q_weight,
+                                                                 q_weight ? head_inv[h] : 1.f, neighbours != 0));
   }
   if (k_col < 0) return;
   const int b = req_of_row[r];
@@ -63,7 +86,8 @@ __global__ void __launch_bounds__(128) qkv_rotate_store_kernel(
   const long long at = (long long)page * Hk * page_size + pos % page_size;
   for (int e = threadIdx.x; e < Hk * D; e += blockDim.x) {
     const int h = e / D, i = e - h * D;
-    k_cache[(at + (long long)h * page_size) * D + i] = from_f32<T>(rotated_entry(row + k_col + h * D, i, half, sn, cs));
+    k_cache[(at + (long long)h * page_size) * D + i] = from_f32<T>(rotated_entry(row + k_col + h * D, i, half, sn, cs, k_weight,
+                                                                                  k_weight ? head_inv[Hq + h] : 1.f, neighbours != 0));
   }
   if (v_other) {
     // blended in 32-bit from the two stored values, rounded once; a blended value is not turned as well
@@ -87,7 +111,8 @@ __global__ void __launch_bounds__(128) attention_flex_kernel(
     const int* __restrict__ block_table, int max_pages, int page_size, int num_pages, const int* __restrict__ req_of_row,
     const int* __restrict__ positions, float scale, float softcap, int window, int keep_first,
     const float* __restrict__ inv_freq_out, const T* __restrict__ gate, long long ld_gate, float out_scale,
-    T* __restrict__ out, long long ld_out, int Hq, int Hk, int D, int VD, int* __restrict__ status) {
+    T* __restrict__ out, long long ld_out, int Hq, int Hk, int D, int VD, int* __restrict__ status, int chunk,
+    const float* __restrict__ sinks, int gate_heads) {
   __shared__ float qs[4][FLEX_MAX_DIM];
   __shared__ float os[4][FLEX_MAX_DIM];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -101,7 +126,7 @@ __global__ void __launch_bounds__(128) attention_flex_kernel(
   for (int i = lane; i < D; i += 32) qv[i] = to_f32(qrow[i]) * scale;
   __syncwarp();
 
-  const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+  const int lo = chunk > 0 ? pos - pos % chunk : (window > 0 ? max(0, pos - window + 1) : 0);
   const int first_end = min(keep_first, lo);        // the kept first tokens that the window does not hold anyway
   constexpr int NACC = FLEX_MAX_DIM / 32;
   float acc[NACC];
@@ -151,7 +176,11 @@ __global__ void __launch_bounds__(128) attention_flex_kernel(
       m = m_new;
     }
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  float inv = l > 0.f ? 1.f / l : 0.f;
+  if (sinks) {            // as one more key that has no value
+    const float top = fmaxf(m, sinks[h]), f = expf(m - top);
+    inv = f / fmaf(l, f, expf(sinks[h] - top));
+  }
   float* ov = os[warp];
 #pragma unroll
   for (int t = 0; t < NACC; ++t) {
@@ -160,7 +189,7 @@ __global__ void __launch_bounds__(128) attention_flex_kernel(
   }
   __syncwarp();
   T* o = out + (long long)r * ld_out + (long long)h * VD;
-  const T* g = gate ? gate + (long long)r * ld_gate + (long long)h * VD : nullptr;
+  const T* g = gate ? gate + (long long)r * ld_gate + (gate_heads ? h : (long long)h * VD) : nullptr;
   const int vhalf = inv_freq_out ? VD / 2 : 0;
   for (int i = lane; i < VD; i += 32) {
     float y = ov[i];
@@ -170,7 +199,7 @@ __global__ void __launch_bounds__(128) attention_flex_kernel(
       sincosf((float)pos * inv_freq_out[f], &sn, &c);
       y = i < vhalf ? ov[i] * c + ov[i + vhalf] * sn : ov[i] * c - ov[i - vhalf] * sn;
     }
-    if (g) y *= 1.f / (1.f + expf(-to_f32(g[i])));
+    if (g) y *= 1.f / (1.f + expf(-to_f32(g[gate_heads ? 0 : i])));
     o[i] = from_f32<T>(y * out_scale);
   }
 }
@@ -184,21 +213,24 @@ extern "C" int tl_qkv_rotate_store(const void* qkv, long long ld, int q_col, int
                                    const int* block_table, int max_pages, int page_size, int num_pages, void* q_out,
                                    void* k_cache, void* v_cache, int rows, int Hq, int Hk, int D, int VD, int dtype,
                                    int* status, float rot_magnitude, const void* v_other, long long ld_other,
-                                   const float* v_blend, cudaStream_t stream) {
+                                   const float* v_blend, const float* q_weight, const float* k_weight, float norm_eps,
+                                   int neighbours, cudaStream_t stream) {
   if (rows == 0) return 0;
   TL_REQUIRE(!v_other || (v_blend && !inv_freq_v), "qkv_rotate_store: blended values want their weight and are not turned");
   TL_REQUIRE(Hq > 0 && Hk > 0 && D >= 1 && D <= FLEX_MAX_DIM && VD >= 1 && VD <= FLEX_MAX_DIM,
              "qkv_rotate_store: %d query heads, %d KV heads, key size %d, value size %d (sizes up to %d)", Hq, Hk, D, VD,
              FLEX_MAX_DIM);
   TL_REQUIRE(!inv_freq || (rot > 0 && rot <= D && rot % 2 == 0), "qkv_rotate_store: rotary size %d for head size %d", rot, D);
+  TL_REQUIRE((q_weight != nullptr) == (k_weight != nullptr) && (!q_weight || Hq + Hk <= 8192),
+             "qkv_rotate_store: norms of q and k come together, for up to 8192 heads");
   TL_REQUIRE(!inv_freq_v || VD % 2 == 0, "qkv_rotate_store: values of odd size %d cannot be turned in pairs", VD);
   TL_REQUIRE(k_col < 0 || (k_cache && v_cache && block_table && page_size > 0 && max_pages > 0),
              "qkv_rotate_store: keys and values without pages to go to");
 #define TL_QRS(T_)                                                                                                         \
-  qkv_rotate_store_kernel<T_><<<rows, 128, 0, stream>>>((const T_*)qkv, ld, q_col, k_col, v_col, inv_freq, rot, inv_freq_v,  \
+  qkv_rotate_store_kernel<T_><<<rows, 128, q_weight ? (Hq + Hk) * sizeof(float) : 0, stream>>>((const T_*)qkv, ld, q_col, k_col, v_col, inv_freq, rot, inv_freq_v,  \
                                                         positions, req_of_row, block_table, max_pages, page_size, num_pages, \
                                                         (T_*)q_out, (T_*)k_cache, (T_*)v_cache, Hq, Hk, D, VD, status,    \
-                                                        rot_magnitude, (const T_*)v_other, ld_other, v_blend)
+                                                        rot_magnitude, (const T_*)v_other, ld_other, v_blend, q_weight, k_weight, norm_eps, neighbours)
   if (dtype == TL_FP32) TL_QRS(float);
   else TL_QRS(bf16);
 #undef TL_QRS
@@ -210,7 +242,8 @@ extern "C" int tl_attention_flex(const void* q, const void* k_cache, const void*
                                  int max_pages, int page_size, int num_pages, const int* req_of_row, const int* positions,
                                  float scale, float softcap, int window, int keep_first, const float* inv_freq_out,
                                  const void* gate, long long ld_gate, float out_scale, void* out, long long ld_out, int rows,
-                                 int Hq, int Hk, int D, int VD, int dtype, int* status, cudaStream_t stream) {
+                                 int Hq, int Hk, int D, int VD, int dtype, int* status, int chunk, const float* sinks, int gate_heads,
+                                 cudaStream_t stream) {
   if (rows == 0) return 0;
   TL_REQUIRE(Hq > 0 && Hk > 0 && Hq % Hk == 0, "attention_flex: %d query heads over %d KV heads", Hq, Hk);
   TL_REQUIRE(D >= 1 && D <= FLEX_MAX_DIM && VD >= 1 && VD <= FLEX_MAX_DIM, "attention_flex: key size %d, value size %d (up to %d)",
@@ -218,6 +251,8 @@ extern "C" int tl_attention_flex(const void* q, const void* k_cache, const void*
   TL_REQUIRE(page_size > 0 && max_pages > 0 && window >= 0 && keep_first >= 0,
              "attention_flex: page size %d, table width %d, window %d, kept first tokens %d", page_size, max_pages, window,
              keep_first);
+  TL_REQUIRE(chunk >= 0 && (chunk == 0 || (window == 0 && keep_first == 0)), "attention_flex: chunks of %d do not combine with a window",
+             chunk);
   TL_REQUIRE(!inv_freq_out || VD % 2 == 0, "attention_flex: outputs of odd size %d cannot be turned in pairs", VD);
   dim3 grid(rows, ceil_div(Hq, 4));
   TL_REQUIRE(grid.y <= 65535, "attention_flex: %d heads exceed the grid limit", Hq);
@@ -225,7 +260,7 @@ extern "C" int tl_attention_flex(const void* q, const void* k_cache, const void*
   attention_flex_kernel<T_><<<grid, 128, 0, stream>>>((const T_*)q, (const T_*)k_cache, (const T_*)v_cache, block_table,     \
                                                       max_pages, page_size, num_pages, req_of_row, positions, scale, softcap, \
                                                       window, keep_first, inv_freq_out, (const T_*)gate, ld_gate, out_scale,   \
-                                                      (T_*)out, ld_out, Hq, Hk, D, VD, status)
+                                                      (T_*)out, ld_out, Hq, Hk, D, VD, status, chunk, sinks, gate_heads)
   if (dtype == TL_FP32) TL_AF(float);
   else TL_AF(bf16);
 #undef TL_AF

@@ -2,9 +2,10 @@
 // design may combine, for prompt portions and for decoding; keys of 64 or 128 entries and, separately, values of 64 or 128.
 //
 //   score = scale q.k, optionally capped (c tanh(score / c)); the row at position i sees key j <= i when there is no
-//   window, or i - j < window, or j < keep_first; softmax in 32-bit; o = a v; the output optionally turned back by the
+//   window, or i - j < window, or j < keep_first, or, with chunks, when i and j lie in the same chunk of positions; softmax in
+//   32-bit, its denominator optionally with exp(sink) of a number a head; o = a v; the output optionally turned back by the
 //   row's own position (halves layout: entry m with entry m + VD / 2, by -i f_m), optionally times sigmoid(gate) entry by
-//   entry, times `out_scale`; written to rows of `ld_out` entries (a column slice of a wider tensor will do)
+//   entry or head by head, times `out_scale`; written to rows of `ld_out` entries (a column slice of a wider tensor will do)
 //
 // One CTA of four warps takes a tile of query rows of one request and one KV head. The G query heads of that KV head are
 // packed into the tile's 64 M rows (M row m = query row m / G, head m % G), so keys and values are read once for the whole
@@ -74,6 +75,9 @@ struct Options {
   const float* inv_freq_out;      // [VD / 2] or null
   const bf16* gate;               // [rows, ld_gate], entry h * VD + i, or null
   long long ld_gate, ld_out;
+  int chunk;                      // > 0: the chunk's positions instead of a window
+  int gate_heads;                 // the gate has one entry a head, gate[row, h]
+  const float* sinks;             // [Hq] or null
 };
 
 template <int D, int VD, bool KEYSPLIT, int STAGES>
@@ -103,7 +107,9 @@ __global__ void __launch_bounds__(128) attention_flex_mma_kernel(
   const int pos0 = positions[row0];
   const int* table = block_table + (long long)b * max_pages;
   // keys any row of the tile may see: the window's k_lo .. k_hi, and the kept first ones below k_lo
-  const int k_lo = window > 0 ? max(0, pos0 - window + 1) : 0;
+  const int chunk = opt.chunk;
+  auto first_seen = [&](int pos) { return chunk > 0 ? pos - pos % chunk : (window > 0 ? max(0, pos - window + 1) : 0); };
+  const int k_lo = first_seen(pos0);
   const int k_hi = pos0 + nq - 1;
   const int first_end = min(keep_first, k_lo);
   const int kt_first = k_lo / KT, kt_last = k_hi / KT;
@@ -172,7 +178,7 @@ __global__ void __launch_bounds__(128) attention_flex_mma_kernel(
   const int q_lo = r_lo / G, q_hi = r_hi / G;
   const bool v_lo = q_lo < nq, v_hi = q_hi < nq;
   const int p_lo = pos0 + q_lo, p_hi = pos0 + q_hi;
-  const int w_lo = window > 0 ? max(0, p_lo - window + 1) : 0, w_hi = window > 0 ? max(0, p_hi - window + 1) : 0;
+  const int w_lo = first_seen(p_lo), w_hi = first_seen(p_hi);
   const int n_base = KEYSPLIT ? warp * 2 : 0;      // first 8-key score tile of this warp
   constexpr float LOG2E = 1.4426950408889634f;
   const float scale = opt.scale, cap = opt.softcap, inv_cap = cap > 0.f ? 1.f / cap : 0.f;
@@ -288,10 +294,15 @@ __global__ void __launch_bounds__(128) attention_flex_mma_kernel(
 
   // Four finished entries of M row r (entries c, c + 1 and their partners VD / 2 further on; c < VD / 2, even): divided by
   // the row's sum, turned back, gated, scaled, written.
-  auto emit = [&](int r, int c, float a0, float a1, float b0, float b1, float l) {
+  // (`m`: the row's maximum in units of log 2, against which the sums were built)
+  auto emit = [&](int r, int c, float a0, float a1, float b0, float b1, float l, float m) {
     const int qi = r / G, head = g * G + r % G;
     const long long row = row0 + qi;
-    const float inv = l > 0.f ? 1.f / l : 0.f;
+    float inv = l > 0.f ? 1.f / l : 0.f;
+    if (opt.sinks) {          // as one more key that has no value
+      const float sink = opt.sinks[head] * LOG2E, top = fmaxf(m, sink), f = exp2f(m - top);
+      inv = f / fmaf(l, f, exp2f(sink - top));
+    }
     a0 *= inv;
     a1 *= inv;
     b0 *= inv;
@@ -308,7 +319,13 @@ __global__ void __launch_bounds__(128) attention_flex_mma_kernel(
       a1 = x1;
       b1 = y1;
     }
-    if (opt.gate) {
+    if (opt.gate && opt.gate_heads) {
+      const float ga = 1.f / (1.f + expf(-to_f32(opt.gate[row * opt.ld_gate + head])));
+      a0 *= ga;
+      a1 *= ga;
+      b0 *= ga;
+      b1 *= ga;
+    } else if (opt.gate) {
       const bf16* gr = opt.gate + row * opt.ld_gate + (long long)head * VD;
       a0 *= 1.f / (1.f + expf(-to_f32(gr[c])));
       a1 *= 1.f / (1.f + expf(-to_f32(gr[c + 1])));
@@ -329,7 +346,7 @@ __global__ void __launch_bounds__(128) attention_flex_mma_kernel(
 #pragma unroll
       for (int n = 0; n < VD / 16; ++n)
         emit(r, n * 8 + (lane & 3) * 2, o[n][half * 2], o[n][half * 2 + 1], o[n + VD / 16][half * 2],
-             o[n + VD / 16][half * 2 + 1], l);
+             o[n + VD / 16][half * 2 + 1], l, half ? m_hi : m_lo);
     }
   } else {
     // ---- merge the four warps' shares of the keys, in warp order ----
@@ -372,7 +389,7 @@ __global__ void __launch_bounds__(128) attention_flex_mma_kernel(
         b1 += f * src[c + VD / 2 + 1];
       }
       if (n_cta == 1) {
-        emit(r, c, a0, a1, b0, b1, l);
+        emit(r, c, a0, a1, b0, b1, l, mrow);
       } else {
         co[r * VD + c] = a0;
         co[r * VD + c + 1] = a1;
@@ -404,7 +421,7 @@ __global__ void __launch_bounds__(128) attention_flex_mma_kernel(
             b0 += f * ld_cluster(co + r * VD + c + VD / 2, w);
             b1 += f * ld_cluster(co + r * VD + c + VD / 2 + 1, w);
           }
-          emit(r, c, a0, a1, b0, b1, l);
+          emit(r, c, a0, a1, b0, b1, l, mrow);
         }
       }
       cluster_sync();        // nobody leaves while its shared memory may still be read
@@ -479,21 +496,26 @@ extern "C" int tl_attention_flex_mma(const void* q, const void* k_cache, const v
                                      int max_tile_rows, const int* positions, float scale, float softcap, int window,
                                      int keep_first, const float* inv_freq_out, const void* gate, long long ld_gate,
                                      float out_scale, void* out, long long ld_out, int rows, int Hq, int Hk, int D, int VD,
-                                     int max_context, int sm_count, int* status, cudaStream_t stream) {
+                                     int max_context, int sm_count, int* status, int chunk, const float* sinks, int gate_heads,
+                                     cudaStream_t stream) {
   if (rows == 0 || n_tiles == 0) return 0;
   TL_REQUIRE(tl_attention_flex_mma_supported(Hq, Hk, D, VD), "attention (tensor cores): %d heads over %d KV heads, keys of %d, values of %d",
              Hq, Hk, D, VD);
   TL_REQUIRE(page_size > 0 && max_pages > 0 && window >= 0 && keep_first >= 0,
              "attention: page size %d, table width %d, window %d, kept first tokens %d", page_size, max_pages, window, keep_first);
+  TL_REQUIRE(chunk >= 0 && (chunk == 0 || (window == 0 && keep_first == 0)), "attention: chunks of %d do not combine with a window",
+             chunk);
   TL_REQUIRE(Hk <= 65535, "attention: %d KV heads exceed the grid limit", Hk);
   TL_REQUIRE(max_tile_rows >= 1 && max_tile_rows <= tl_attention_flex_mma_tile_rows(Hq, Hk),
              "attention: tiles of %d query rows, at most %d fit", max_tile_rows, tl_attention_flex_mma_tile_rows(Hq, Hk));
   TL_REQUIRE(((uintptr_t)out % 4) == 0 && ld_out % 2 == 0, "attention: output rows of %lld entries must start on 4 bytes", ld_out);
-  fx::Options opt{scale, softcap, out_scale, window, keep_first, inv_freq_out, (const bf16*)gate, ld_gate, ld_out};
+  fx::Options opt{scale, softcap, out_scale, window, keep_first, inv_freq_out, (const bf16*)gate, ld_gate, ld_out, chunk, gate_heads,
+                  sinks};
   const bool keysplit = max_tile_rows * (Hq / Hk) <= 16;
   int cluster = 1;
   if (keysplit) {
-    const int reach = window > 0 ? (max_context < window + keep_first + fx::KT ? max_context : window + keep_first + fx::KT) : max_context;
+    const int reach = chunk > 0 ? (max_context < chunk + fx::KT ? max_context : chunk + fx::KT)
+                      : window > 0 ? (max_context < window + keep_first + fx::KT ? max_context : window + keep_first + fx::KT) : max_context;
     const int key_tiles = (reach + fx::KT - 1) / fx::KT;
     const long long ctas = (long long)n_tiles * Hk;
     while (cluster < 8 && 2 * cluster <= key_tiles && ctas * cluster < (sm_count > 0 ? sm_count : 148)) cluster *= 2;

@@ -169,6 +169,8 @@ __device__ __forceinline__ float gate_activation(float g, int act) {
     default: return g / (1.f + expf(-g));
   }
 }
+// The same code negated is how a launcher of gated products is asked for the ungated form: W holds N rows a group and the plain
+// product's result goes through the activation, C = act(X W^T).
 // An activation with up to two constants of its own (`a0`, `a1`; the codes above that have none ignore them).
 __device__ __forceinline__ float activation(float z, int act, float a0, float a1) {
   if (act == TL_ACT_XIELU) return z > 0.f ? fmaf(a0 * z, z, 0.5f * z) : fmaf(a1, expm1f(z) - z, 0.5f * z);

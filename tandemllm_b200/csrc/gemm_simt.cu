@@ -31,6 +31,7 @@ struct GemmParams {
   int a_div;
   float ga0, ga1;          // the constants of a gate form that has some
   int swiglu;              // a gate activation TL_ACT_* (1: SiLU): W holds 2 N rows per group; C = act(A W[0:N]^T) * (A W[N:2N]^T)
+                           // (negative: N rows per group, C = act(A W^T) with the code's activation; grouped products only)
 };
 
 template <typename TIn, typename TOut, bool SWIGLU>
@@ -126,6 +127,7 @@ __global__ void __launch_bounds__(256) gemm_tiled_kernel(GemmParams p) {
         v = gated(v, acc2[i][j], p.swiglu, p.ga0, p.ga1);
       } else {
         if (p.bias) v += p.bias[n];
+        if (p.swiglu < 0) v = gate_activation(v, -p.swiglu);
       }
       C[r * p.ldc + n] = from_f32<TOut>(v);
     }
@@ -248,7 +250,7 @@ static int launch(const GemmParams& p, int max_tiles, cudaStream_t stream) {
     return 0;
   }
   dim3 grid(ceil_div(p.N, BN), p.tile_group ? max_tiles : ceil_div(p.M, BM));
-  if (p.swiglu)
+  if (p.swiglu > 0)
     gemm_tiled_kernel<TIn, TOut, true><<<grid, 256, 0, stream>>>(p);
   else
     gemm_tiled_kernel<TIn, TOut, false><<<grid, 256, 0, stream>>>(p);

@@ -265,7 +265,7 @@ __global__ void __launch_bounds__(SKINNY_WARPS * 32) gemm_skinny_grouped_kernel(
 #pragma unroll
       for (int s = 0; s < SKINNY_WARPS; ++s) v[j] += part[s][j][row][m];
     }
-    const float r = SWIGLU ? gated(v[0], v[W_TILES - 1], act, ga0, ga1) : v[0];
+    const float r = SWIGLU ? gated(v[0], v[W_TILES - 1], act, ga0, ga1) : (act < 0 ? gate_activation(v[0], -act) : v[0]);
     out[(long long)s_pair[m] * ldc + n0 + row] = from_f32<TOut>(r);
   }
 }
@@ -445,7 +445,7 @@ extern "C" int tl_gemm_skinny_mma(const void* x, long long ldx, const void* w, l
 }
 
 // The routed experts of a very small step. x [*, K] bfloat16; w [groups * rows_per_group, K] bfloat16 with, per group, N
-// rows (or, with swiglu, which is then the gate's activation TL_ACT_*, N gate rows then N up rows); the plan's tiles hold at most 8 rows; out [pairs, N] in the plan's
+// rows (or, with swiglu, which is then the gate's activation TL_ACT_*, N gate rows then N up rows; negated: N rows whose results go through the activation); the plan's tiles hold at most 8 rows; out [pairs, N] in the plan's
 // order, bfloat16 or 32-bit. row_index (or null) and row_div as in the kernel's comment.
 extern "C" int tl_gemm_skinny_grouped(const void* x, long long ldx, const int* row_index, int row_div, const void* w,
                                       long long ldw, long long rows_per_group, void* out, long long ldc, int N, int K,
@@ -461,14 +461,14 @@ extern "C" int tl_gemm_skinny_grouped(const void* x, long long ldx, const int* r
                              : (tile_group && tile_row0 && tile_rows && n_tiles)),
              "skinny grouped product: operands must be 16-byte aligned and the plan complete, or at most %d pairs given",
              SKINNY_WARPS * 32);
-  TL_REQUIRE(swiglu >= 0 && swiglu <= TL_ACT_GATE_LAST, "skinny grouped product: gate activation %d is not one of 0..%d", swiglu,
-             TL_ACT_GATE_LAST);
+  TL_REQUIRE(swiglu >= -TL_ACT_IDENTITY && swiglu <= TL_ACT_GATE_LAST,
+             "skinny grouped product: gate activation %d is not one of 0..%d (or an ungated one, negated)", swiglu, TL_ACT_GATE_LAST);
   const dim3 grid(ceil_div(N, 16), max_tiles), block(SKINNY_WARPS * 32);
 #define TL_GROUPED(SW_, T_)                                                                                              \
   return (int)launch_chained(gemm_skinny_grouped_kernel<SW_, T_>, grid, block, 0, stream, (const bf16*)x, ldx, row_index,  \
                              row_div, (const bf16*)w, ldw, rows_per_group, (T_*)out, ldc, N, K, tile_group, tile_row0,    \
                              tile_rows, n_tiles, pair_group, n_pairs, n_groups, status, swiglu, tl_gate_constants[0], tl_gate_constants[1], 0u)
-  if (swiglu) {
+  if (swiglu > 0) {
     if (out_dtype == TL_FP32) TL_GROUPED(true, float);
     TL_GROUPED(true, bf16);
   }

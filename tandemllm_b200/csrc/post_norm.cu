@@ -150,6 +150,62 @@ __global__ void __launch_bounds__(256) add_normed_kernel(PostNormParams p) {
   for (int c = threadIdx.x; c < hidden; c += blockDim.x) out[c] = from_f32<T>(row[c] * inv2 * p.pre_weight[c]);
 }
 
+// out[r] = scale * (weight_a * a[r] / rms(a[r]) + weight_b * b[r] / rms(b[r])): two branches' rows, each normed on its own (a tensor or
+// partial sums each, added in order). One block a row.
+struct NormedSumParams {
+  const float *a, *b;
+  int a_parts, b_parts;
+  long long part_stride;
+  const float *weight_a, *weight_b;
+  float eps, scale;
+  float* out;
+  int hidden;
+};
+template <int CPT>
+__global__ void __launch_bounds__(256) normed_sum_kernel(NormedSumParams p) {
+  __shared__ float scratch[33];
+  const int hidden = p.hidden;
+  const size_t at = (size_t)blockIdx.x * hidden;
+  float a[CPT], b[CPT];
+  float sa = 0.f, sb = 0.f;
+#pragma unroll
+  for (int i = 0; i < CPT; ++i) {
+    const int c = threadIdx.x + i * blockDim.x;
+    a[i] = c < hidden ? p.a[at + c] : 0.f;
+    b[i] = c < hidden ? p.b[at + c] : 0.f;
+  }
+  for (int s = 1; s < p.a_parts; ++s) {
+    const float* src = p.a + (long long)s * p.part_stride + at;
+#pragma unroll
+    for (int i = 0; i < CPT; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c < hidden) a[i] += src[c];
+    }
+  }
+  for (int s = 1; s < p.b_parts; ++s) {
+    const float* src = p.b + (long long)s * p.part_stride + at;
+#pragma unroll
+    for (int i = 0; i < CPT; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c < hidden) b[i] += src[c];
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < CPT; ++i) {
+    sa = fmaf(a[i], a[i], sa);
+    sb = fmaf(b[i], b[i], sb);
+  }
+  sa = block_sum(sa, scratch);
+  __syncthreads();
+  sb = block_sum(sb, scratch);
+  const float ia = rsqrtf(sa / (float)hidden + p.eps), ib = rsqrtf(sb / (float)hidden + p.eps);
+#pragma unroll
+  for (int i = 0; i < CPT; ++i) {
+    const int c = threadIdx.x + i * blockDim.x;
+    if (c < hidden) p.out[at + c] = p.scale * (a[i] * ia * p.weight_a[c] + b[i] * ib * p.weight_b[c]);
+  }
+}
+
 // out[r] = x[r, :] . w: a warp a row (a projection onto one number a row, such as the logit of a gate)
 template <typename T>
 __global__ void __launch_bounds__(256) row_dot_kernel(const T* __restrict__ x, long long ld_x, const T* __restrict__ w,
@@ -208,6 +264,22 @@ extern "C" int tl_add_normed(float* residual, const float* delta, int parts, lon
     else TL_ADD_NORMED(bf16, false);
   }
 #undef TL_ADD_NORMED
+  TL_LAUNCH_CHECK();
+  return 0;
+}
+
+extern "C" int tl_normed_sum(const float* a, int a_parts, const float* b, int b_parts, long long part_stride, const float* weight_a,
+                             const float* weight_b, float eps, float scale, float* out, int rows, int hidden, cudaStream_t stream) {
+  if (rows == 0) return 0;
+  TL_REQUIRE(rows > 0 && hidden > 0 && hidden <= 16384 && a && b && a_parts >= 1 && b_parts >= 1, "normed_sum: %d rows of %d", rows,
+             hidden);
+  NormedSumParams p{a, b, a_parts, b_parts, part_stride, weight_a, weight_b, eps, scale, out, hidden};
+  const int threads = hidden <= 512 ? 64 : (hidden <= 1024 ? 128 : 256);
+  const int cpt = ceil_div(hidden, threads);
+  if (cpt <= 8) normed_sum_kernel<8><<<rows, threads, 0, stream>>>(p);
+  else if (cpt <= 16) normed_sum_kernel<16><<<rows, threads, 0, stream>>>(p);
+  else if (cpt <= 32) normed_sum_kernel<32><<<rows, threads, 0, stream>>>(p);
+  else normed_sum_kernel<64><<<rows, threads, 0, stream>>>(p);
   TL_LAUNCH_CHECK();
   return 0;
 }

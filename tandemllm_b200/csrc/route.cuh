@@ -4,9 +4,11 @@
 // Ties go to the lower expert id; a NaN score is chosen only when nothing else is left.
 // (engine/models/lfm2_moe/ref.py:185-197, engine/models/lfm2_moe/kernels.py:265-287 of the reference; the softmax
 // scoring is what its other routed families use, engine/models/flashnext/ref.py:479-487)
+// The third scoring function takes the bias as part of the logit: the k largest logits + bias are chosen, and their weights are
+// the softmax over the chosen ones only (computed from the row's largest logit, which is always chosen).
 //
 // The launchers' `normalize` argument carries the router's choices: bit 0 = divide the chosen weights by their sum,
-// bits 1..3 = the scoring function (TL_SCORE_SIGMOID 0, TL_SCORE_SOFTMAX 1), bits 4..9 = the number of expert groups
+// bits 1..3 = the scoring function (TL_SCORE_SIGMOID 0, TL_SCORE_SOFTMAX 1, TL_SCORE_CHOSEN 2), bits 4..9 = the number of expert groups
 // (0: the choice is free) and bits 10..15 = how many of them are kept.
 //
 // Group-limited choice: the experts form `groups` equal groups of neighbours; a group's score is the sum of its two
@@ -20,7 +22,8 @@ namespace tl {
 
 #define TL_SCORE_SIGMOID 0
 #define TL_SCORE_SOFTMAX 1
-#define TL_SCORE_LAST 1
+#define TL_SCORE_CHOSEN 2
+#define TL_SCORE_LAST 2
 #define TL_ROUTE_SCORING(flags) (((flags) >> 1) & 7)
 #define TL_ROUTE_GROUPS(flags) (((flags) >> 4) & 63)
 #define TL_ROUTE_KEEP(flags) (((flags) >> 10) & 63)
@@ -38,6 +41,10 @@ __device__ __forceinline__ void warp_route_sized(const float* lg, const float* _
   const int scoring = TL_ROUTE_SCORING(normalize);
   const int n_groups = TL_ROUTE_GROUPS(normalize), keep_groups = TL_ROUTE_KEEP(normalize);
   normalize &= 1;
+  if (scoring == TL_SCORE_CHOSEN) {
+    normalize = 1;
+    floor_ = 0.f;
+  }
   float score[PER], choice[PER];
   float top = -INFINITY, denom = 1.f;
   if (scoring == TL_SCORE_SOFTMAX) {        // the row's largest logit and the sum of exponentials, over the whole warp
@@ -51,13 +58,26 @@ __device__ __forceinline__ void warp_route_sized(const float* lg, const float* _
       if (lane + 32 * t < E) part += expf(lg[lane + 32 * t] - top);
     denom = warp_sum(part);
   }
+  if (scoring == TL_SCORE_CHOSEN) {
+#pragma unroll
+    for (int t = 0; t < PER; ++t) {
+      const int e = lane + 32 * t;
+      if (e < E) top = fmaxf(top, bias ? lg[e] + bias[e] : lg[e]);
+    }
+    top = warp_max(top);
+  }
 #pragma unroll
   for (int t = 0; t < PER; ++t) {
     const int e = lane + 32 * t;
     if (e < E) {
-      const float s = scoring == TL_SCORE_SOFTMAX ? expf(lg[e] - top) / denom : 1.f / (1.f + expf(-lg[e]));
-      score[t] = s;
-      choice[t] = bias ? s + bias[e] : s;
+      if (scoring == TL_SCORE_CHOSEN) {
+        choice[t] = bias ? lg[e] + bias[e] : lg[e];
+        score[t] = expf(choice[t] - top);
+      } else {
+        const float s = scoring == TL_SCORE_SOFTMAX ? expf(lg[e] - top) / denom : 1.f / (1.f + expf(-lg[e]));
+        score[t] = s;
+        choice[t] = bias ? s + bias[e] : s;
+      }
       if (!(choice[t] == choice[t])) choice[t] = -INFINITY;
     } else {
       score[t] = 0.f;

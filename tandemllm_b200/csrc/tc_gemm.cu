@@ -46,7 +46,8 @@ struct TcParams {
   const int* n_tiles;
   const int* row_index;       // grouped, swapped: token row of sorted position i is row_index[i] / row_div of X (or nullptr:
   int row_div;                // X is already in sorted order)
-  int act;                    // the gate's activation of a gated product (TL_ACT_*), 0 for a plain one
+  int act;                    // the gate's activation of a gated product (TL_ACT_*), 0 for a plain one; negated: an activation
+                              // on a plain product's results
   float ga0, ga1;             // the constants of a gate form that has some
   int skip_kb;                // -1; a test sets the k-block whose copies the producer leaves out, so that a wait runs out
   int* status;
@@ -102,6 +103,8 @@ __device__ __forceinline__ void tmem_ld16(uint32_t taddr, float* v) {
 template <typename TOut> __device__ __forceinline__ void store_out(TOut* p, float v);
 template <> __device__ __forceinline__ void store_out<float>(float* p, float v) { *p = v; }
 template <> __device__ __forceinline__ void store_out<bf16>(bf16* p, float v) { *p = __float2bfloat16_rn(v); }
+
+__device__ __forceinline__ float plain_result(float v, int act) { return act < 0 ? gate_activation(v, -act) : v; }
 
 template <int BN, bool SWAP, bool SWIGLU>
 struct Smem {
@@ -312,7 +315,7 @@ __global__ void __launch_bounds__(192) gemm_tc_kernel(const __grid_constant__ CU
             for (int j = 0; j < 16; ++j) {
               const int t = c0 + j;
               if (t < tok_rows) {
-                const float r = SWIGLU ? gated(v[j], u[j], p.act, p.ga0, p.ga1) : v[j] + b;
+                const float r = SWIGLU ? gated(v[j], u[j], p.act, p.ga0, p.ga1) : plain_result(v[j] + b, p.act);
                 if (p.partial) p.partial[((long long)blockIdx.z * p.M + tok0 + t) * p.N + n] = r;
                 else store_out<TOut>(C + (long long)(tok0 + t) * p.ldc + n, r);
               }
@@ -326,7 +329,8 @@ __global__ void __launch_bounds__(192) gemm_tc_kernel(const __grid_constant__ CU
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
               const int n = n0 + c0 + j;
-              r[j] = SWIGLU ? gated(v[j], u[j], p.act, p.ga0, p.ga1) : v[j] + ((p.bias && n < p.N) ? p.bias[n] : 0.f);
+              r[j] = SWIGLU ? gated(v[j], u[j], p.act, p.ga0, p.ga1)
+                            : plain_result(v[j] + ((p.bias && n < p.N) ? p.bias[n] : 0.f), p.act);
             }
             // 16 consecutive outputs of one row: 16-byte stores when they are all there and aligned
             const bool whole = n0 + c0 + 16 <= p.N && (((uintptr_t)(row + n0 + c0)) & 15) == 0;
@@ -535,7 +539,8 @@ __global__ void __launch_bounds__(192) gemm_tc_persistent_kernel(const __grid_co
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
             const int col = n0 + c0 + j;
-            r[j] = SWIGLU ? gated(v[j], u[j], p.act, p.ga0, p.ga1) : v[j] + ((p.bias && col < p.N) ? p.bias[col] : 0.f);
+            r[j] = SWIGLU ? gated(v[j], u[j], p.act, p.ga0, p.ga1)
+                          : plain_result(v[j] + ((p.bias && col < p.N) ? p.bias[col] : 0.f), p.act);
           }
           const bool whole = n0 + c0 + 16 <= p.N && (((uintptr_t)(row + n0 + c0)) & 15) == 0;
           if (whole) {
@@ -669,7 +674,7 @@ extern "C" int tl_tc_token_tile(int swap, int bn) { return swap ? bn : TILE_M; }
 // 128 up rows with swiglu).
 
 // X [M, K] (row stride ldx), W [groups * rows_per_group, K] (row stride ldw). Plain: groups = 1, tile_group = nullptr.
-// swiglu: W holds 2 N rows per group (gate then up) and C = silu(gate) * up. out_dtype: TL_BF16 or TL_FP32.
+// swiglu: W holds 2 N rows per group (gate then up) and C = act(gate) * up; a negated code: N rows and C = act(X W^T). out_dtype: TL_BF16 or TL_FP32.
 // splits > 1 (swap, not swiglu): `partial` must hold splits * M * N floats; a grouped product leaves the sums to the caller.
 // row_index (swap, grouped; or null): the tile map's rows are positions of this list, and position i stands for row
 // row_index[i] / row_div of X; without it X itself is in the tile map's order.
@@ -687,8 +692,10 @@ extern "C" int tl_gemm_tc(const void* X, long long ldx, long long x_rows, const 
   TL_REQUIRE(out_dtype == TL_BF16 || out_dtype == TL_FP32, "tensor-core gemm: output dtype %d", out_dtype);
   TL_REQUIRE(splits >= 1 && (splits == 1 || (swap && !swiglu && partial && (!tile_group || !reduce))),
              "tensor-core gemm: split-K needs the swapped plain kernel and a workspace (grouped: the caller adds the sums)");
+  const bool gated_form = swiglu > 0;
   TL_REQUIRE(!bias || !swiglu, "tensor-core gemm: a bias with the gated epilogue is not implemented");
-  TL_REQUIRE(swiglu >= 0 && swiglu <= TL_ACT_GATE_LAST, "tensor-core gemm: gate activation %d is not one of 0..%d", swiglu, TL_ACT_GATE_LAST);
+  TL_REQUIRE(swiglu >= -TL_ACT_IDENTITY && swiglu <= TL_ACT_GATE_LAST,
+             "tensor-core gemm: gate activation %d is not one of 0..%d (or an ungated one, negated)", swiglu, TL_ACT_GATE_LAST);
   TL_REQUIRE(!row_index || (swap && tile_group && row_div >= 1),
              "tensor-core gemm: a row index needs the swapped grouped kernel (divisor %d)", row_div);
   CUtensorMap tmW, tmX;
@@ -712,23 +719,23 @@ extern "C" int tl_gemm_tc(const void* X, long long ldx, long long x_rows, const 
   TL_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "tensor-core gemm: grid %u x %u x %u exceeds the limits", grid.x, grid.y, grid.z);
   int e;
   if (persistent) {
-    const int out_n = swiglu ? 128 : 256;
+    const int out_n = gated_form ? 128 : 256;
     const long long work = (long long)ceil_div(N, out_n) * (tile_group ? max_tiles : ceil_div(M, TILE_M));
     const int sms = sm_count();
     const dim3 pgrid((unsigned)(work < sms ? work : sms));
-    if (swiglu) e = out_dtype == TL_BF16 ? launch_persistent<true, bf16>(tmW, tmX, p, pgrid, stream)
+    if (gated_form) e = out_dtype == TL_BF16 ? launch_persistent<true, bf16>(tmW, tmX, p, pgrid, stream)
                                          : launch_persistent<true, float>(tmW, tmX, p, pgrid, stream);
     else e = out_dtype == TL_BF16 ? launch_persistent<false, bf16>(tmW, tmX, p, pgrid, stream)
                                   : launch_persistent<false, float>(tmW, tmX, p, pgrid, stream);
     return e;
   }
   if (swap) {
-    if (swiglu) e = out_dtype == TL_BF16 ? launch_bn<true, true, bf16>(bn, tmW, tmX, p, grid, stream)
+    if (gated_form) e = out_dtype == TL_BF16 ? launch_bn<true, true, bf16>(bn, tmW, tmX, p, grid, stream)
                                          : launch_bn<true, true, float>(bn, tmW, tmX, p, grid, stream);
     else e = out_dtype == TL_BF16 ? launch_bn<true, false, bf16>(bn, tmW, tmX, p, grid, stream)
                                   : launch_bn<true, false, float>(bn, tmW, tmX, p, grid, stream);
   } else {
-    if (swiglu) e = out_dtype == TL_BF16 ? launch_bn<false, true, bf16>(bn, tmW, tmX, p, grid, stream)
+    if (gated_form) e = out_dtype == TL_BF16 ? launch_bn<false, true, bf16>(bn, tmW, tmX, p, grid, stream)
                                          : launch_bn<false, true, float>(bn, tmW, tmX, p, grid, stream);
     else e = out_dtype == TL_BF16 ? launch_bn<false, false, bf16>(bn, tmW, tmX, p, grid, stream)
                                   : launch_bn<false, false, float>(bn, tmW, tmX, p, grid, stream);

@@ -514,7 +514,7 @@ extern "C" int tl_tc_pair_resident(int gated, int per_sm) {
 
 // X [M, K] (row stride ldx, x_rows rows in the tensor), W [groups * rows_per_group, K] (row stride ldw). Plain: groups = 1,
 // tile_group = nullptr. gated (an activation code TL_ACT_*, or 0): W holds 2 N rows per group (gate then up) and
-// C = act(gate) * up. out_dtype: TL_BF16 or TL_FP32. Grouped: the tile map's tiles hold at most tl_tc_pair_token_tile()
+// C = act(gate) * up; a negated code: N rows and C = act(X W^T). out_dtype: TL_BF16 or TL_FP32. Grouped: the tile map's tiles hold at most tl_tc_pair_token_tile()
 // rows (plan_rows: the height the map was built with). per_sm: 1 or 2 CTAs an SM (see Smem). splits > 1 (plain, ungrouped,
 // 32-bit output): the reduction is cut into `splits` runs of k-blocks, each a work item of its own, and C receives the
 // runs' partial results one behind the other, [splits, M, ldc], for the caller to add in order (a product with fewer
@@ -573,8 +573,9 @@ extern "C" int tl_gemm_tc_pair(const void* X, long long ldx, long long x_rows, c
                                int gated, int out_dtype, const int* tile_group, const int* tile_row0, const int* tile_rows,
                                const int* n_tiles, int max_tiles, int plan_rows, int per_sm, int splits, int* status,
                                cudaStream_t stream) {
-  return pair_product(X, ldx, x_rows, W, ldw, w_rows, rows_per_group, bias, C, ldc, M, N, K, gated, out_dtype, tile_group,
-                      tile_row0, tile_rows, n_tiles, max_tiles, plan_rows, per_sm, splits, 0, 0.f, 0.f, status, stream);
+  return pair_product(X, ldx, x_rows, W, ldw, w_rows, rows_per_group, bias, C, ldc, M, N, K, gated > 0 ? gated : 0, out_dtype,
+                      tile_group, tile_row0, tile_rows, n_tiles, max_tiles, plan_rows, per_sm, splits, gated < 0 ? -gated : 0, 0.f,
+                      0.f, status, stream);
 }
 
 // C = act(X W^T + bias): the plain, ungrouped product with an activation (TL_ACT_*, constants a0 and a1) in its epilogue.

@@ -435,7 +435,7 @@ class Engine:
         elem = torch.empty(0, dtype=self.cache.dtype).element_size() if self.cache.groups else 0
         kv = 0
         for g in self.cache.groups:
-            span = context if g.need.window is None else min(context, g.need.window + g.need.keep_first)
+            span = context if g.need.reach is None else min(context, g.need.reach + g.need.keep_first)
             per_token = g.need.head_dim + ((g.need.value_dim or g.need.head_dim) if g.need.values else 0)
             kv += len(g.sites) * g.need.kv_heads * per_token * elem * span * batch
         out["kv"] = kv

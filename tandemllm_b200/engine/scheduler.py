@@ -117,7 +117,7 @@ class Scheduler:
         most = min(n + request.params.max_tokens, self.max_model_len)
         ps = self.cache.page_size
         for g in self.cache.groups:
-            span = most if g.need.window is None else min(most, g.need.window + self.chunk_size + ps + g.need.keep_first)
+            span = most if g.need.reach is None else min(most, g.need.reach + self.chunk_size + ps + g.need.keep_first)
             if -(-span // ps) > g.pool.num_pages:
                 raise ValueError(f"request {request.request_id!r}: {most} tokens need {-(-span // ps)} pages, "
                                  f"the pool has {g.pool.num_pages}")
@@ -145,8 +145,8 @@ class Scheduler:
             for q, total in totals.values():
                 table = g.tables.get(q.request_id, [])
                 more = -(-total // ps) - len(table)
-                if g.need.window is not None:
-                    span = -(-(g.need.window + self.chunk_size + ps + g.need.keep_first) // ps)
+                if g.need.reach is not None:
+                    span = -(-(g.need.reach + self.chunk_size + ps + g.need.keep_first) // ps)
                     more = min(more, span - sum(1 for p in table if p >= 0))
                 need += max(0, more)
             if need > g.pool.free:

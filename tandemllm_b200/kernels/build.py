@@ -34,13 +34,14 @@ NVCC_FLAGS = ["-std=c++17", "-O3", "-lineinfo", "-Xcompiler", "-fPIC", "--expt-r
 
 LIBRARIES: dict[str, list[str]] = {
     # every kernel of the 32-bit path, and the plain bfloat16 variants of the same kernels
-    "core": ["rows.cu", "dyt_act.cu", "gemm_simt.cu", "conv.cu", "attention_simt.cu", "attention_split.cu",
-             "attention_headmix.cu", "attention_latent.cu", "attention_flex.cu", "ssm.cu", "recurrence.cu", "layernorm.cu", "post_norm.cu", "moe_route.cu", "sampling.cu", "graphs.cu"],
+    "core": ["rows.cu", "rows_pair.cu", "dyt_act.cu", "gemm_simt.cu", "conv.cu", "attention_simt.cu", "attention_split.cu",
+             "attention_headmix.cu", "attention_latent.cu", "attention_flex.cu", "ssm.cu", "recurrence.cu", "recurrence_write.cu",
+             "layernorm.cu", "post_norm.cu", "moe_route.cu", "sampling.cu", "graphs.cu"],
     # the tcgen05 / TMA kernels of the bfloat16 path; a 32-bit run never builds or loads them
     "tensorcore": ["tc_gemm.cu", "tc_gemm_pair.cu", "attention_mma.cu", "attention_tc.cu", "attention_headmix_mma.cu",
                    "attention_latent_mma.cu", "attention_flex_mma.cu", "head_linear_mma.cu", "gemm_skinny_mma.cu"],
 }
-HEADERS = ["common.cuh", "route.cuh", "attention_noalloc.h", "tma.cuh"]
+HEADERS = ["common.cuh", "route.cuh", "add_rmsnorm.cuh", "recurrence.cuh", "attention_noalloc.h", "tma.cuh"]
 
 _loaded: dict[str, ctypes.CDLL] = {}
 _lock = threading.Lock()

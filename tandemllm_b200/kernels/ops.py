@@ -19,7 +19,7 @@ TL_BAD_ARGUMENT = 100001
 # the gate activations of gated products (TL_ACT_* of csrc/common.cuh) and the router's scoring functions (TL_SCORE_*
 # of csrc/route.cuh), by the names a part's spec gives them
 ACTIVATIONS = {"silu": 1, "gelu": 2, "relu2": 3, "identity": 4, "xielu": 5, "clamped_swish": 6, "softcap": 7, "tanh": 8, "scale": 9}
-SCORINGS = {"sigmoid": 0, "softmax": 1}
+SCORINGS = {"sigmoid": 0, "softmax": 1, "chosen_softmax": 2}
 
 
 def activation_code(name: str) -> int:
@@ -73,6 +73,11 @@ _SIGNATURES = {
                        c_void_p,
                        c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
                        c_float, c_float, c_void_p, c_void_p, c_void_p],
+    "tl_add_rmsnorm_pair": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_int, c_longlong, c_void_p, c_int, c_longlong, c_void_p,
+                            c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int,
+                            c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p, c_void_p],
+    "tl_normed_sum": [c_void_p, c_int, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_float, c_float, c_void_p, c_int, c_int,
+                      c_void_p],
     "tl_gated_mul": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "tl_gemm_simt": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int,
                      c_int, c_int, c_void_p],
@@ -133,14 +138,23 @@ _SIGNATURES = {
                          c_int, c_void_p],
     "tl_qkv_rotate_store": [c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                             c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                            c_void_p, c_float, c_void_p, c_longlong, c_void_p, c_void_p],
+                            c_void_p, c_float, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p],
     "tl_attention_flex": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_float,
                           c_int, c_int, c_void_p, c_void_p, c_longlong, c_float, c_void_p, c_longlong, c_int, c_int, c_int,
-                          c_int, c_int, c_int, c_void_p, c_void_p],
+                          c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p],
     "tl_recurrence_scan": [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p,
                            c_float, c_float, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int,
                            c_int, c_int, c_void_p, c_longlong, c_int, c_int, c_float, c_void_p],
     "tl_recurrence_scratch_floats": [c_longlong, c_int, c_int, c_int, c_int],
+    "tl_gated_delta_scan": [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_float,
+                            c_float, c_void_p, c_int, c_int, c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_void_p, c_int,
+                            c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_longlong, c_int, c_void_p],
+    "tl_matrix_memory_scan": [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_float, c_void_p,
+                              c_longlong, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+                              c_int, c_void_p, c_longlong, c_int, c_void_p],
+    "tl_write_scan_scratch_floats": [c_longlong, c_int, c_int, c_int, c_int],
+    "tl_memory_norm_gate": [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_float, c_float, c_void_p, c_longlong, c_int, c_int,
+                            c_int, c_int, c_void_p],
     "tl_group_norm_gate": [c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_float, c_float, c_void_p, c_longlong, c_int,
                            c_int, c_int, c_int, c_int, c_int, c_void_p],
     "tl_set_gate_constants": [c_float, c_float],
@@ -170,6 +184,7 @@ def core():
         lib.tl_headmix_scratch_floats.argtypes = [c_int, c_int, c_int, c_int]
         lib.tl_headmix_scratch_floats.restype = c_longlong
         lib.tl_recurrence_scratch_floats.restype = c_longlong
+        lib.tl_write_scan_scratch_floats.restype = c_longlong
         lib.tl_ssm_scan_scratch.argtypes = [c_int, c_int, c_int, c_int, c_int]
         lib.tl_ssm_scan_scratch.restype = c_longlong
         lib.tl_last_error.restype = ctypes.c_char_p
@@ -280,6 +295,18 @@ class GatedSum:
         return total if self.experts is None else total + self.experts.materialize()
 
 
+class BranchSum:
+    """Two branch outputs of one row, `first` + `second`, each None, a tensor or a deferred form (a mixer and a feed-forward that
+    both read the residual as it was): the next norm's kernel adds both."""
+
+    def __init__(self, first, second):
+        self.first, self.second = first, second
+
+    def materialize(self):
+        a, b = materialize(self.first), materialize(self.second)
+        return b if a is None else (a if b is None else a.float() + b.float())
+
+
 class StreamUpdate:
     """What a sublayer leaves for a residual of several streams [streams, rows, hidden] (hyper-connections): its output `delta`
     (None, a tensor or a deferred form) with the weights that take it into the streams, all streams at once from the old
@@ -296,7 +323,7 @@ class StreamUpdate:
 
 def materialize(branch):
     """A branch output as a plain tensor, whatever form a part returned it in."""
-    return branch.materialize() if isinstance(branch, (PartialSums, ExpertRows, GatedSum)) else branch
+    return branch.materialize() if isinstance(branch, (PartialSums, ExpertRows, GatedSum, BranchSum)) else branch
 
 
 def add_rmsnorm(residual: torch.Tensor, delta, weight: torch.Tensor, eps: float, out: torch.Tensor,
@@ -311,6 +338,10 @@ def add_rmsnorm(residual: torch.Tensor, delta, weight: torch.Tensor, eps: float,
     _need(residual, torch.float32, "residual"); _need(weight, torch.float32, "norm weight"); _need(out, None, "normed")
     if out32 is not None:
         _need(out32, torch.float32, "normed32")
+    if isinstance(delta, BranchSum):
+        if out32 is not None:
+            raise KernelError("unrounded rows beside the sum of two branches")
+        return add_rmsnorm_pair(residual, delta, weight, eps, out, None, None, gather, route)
     streams, hc = 0, None
     if isinstance(delta, StreamUpdate):
         hc, delta = delta, delta.delta
@@ -349,6 +380,63 @@ def add_rmsnorm(residual: torch.Tensor, delta, weight: torch.Tensor, eps: float,
         float(r.get("floor", 0.0)), float(r.get("scale", 1.0)), ptr(r.get("ids")), ptr(r.get("wts")),
         streams, residual.stride(0) if streams else 0, ptr(hc.mix) if hc else None, ptr(hc.out) if hc else None,
         ptr(hc.read) if hc else None, stream()), "add_rmsnorm")
+    return out
+
+
+def add_rmsnorm_pair(residual: torch.Tensor, delta, weight: torch.Tensor, eps: float, out: torch.Tensor, weight2: torch.Tensor | None,
+                     out2: torch.Tensor | None, gather: torch.Tensor | None = None, route: dict | None = None) -> torch.Tensor:
+    """residual += delta (None, a branch output in any form, or a `BranchSum` of two); out = weight * row / rms(row) and, with
+    `weight2`, out2 = weight2 * row / rms(row) of the same new row. `gather` and `route` as in `add_rmsnorm`; the router reads
+    the second norm's unrounded rows (the first's without a second)."""
+    _need(residual, torch.float32, "residual"); _need(weight, torch.float32, "norm weight"); _need(out, None, "normed")
+    if residual.dim() != 2:
+        raise KernelError(f"two branches for a residual of shape {tuple(residual.shape)}")
+    if weight2 is not None:
+        _need(weight2, torch.float32, "norm weight"); _need(out2, out.dtype, "normed")
+    dense, experts = [], None
+    for piece in ((delta.first, delta.second) if isinstance(delta, BranchSum) else (delta,)):
+        if isinstance(piece, ExpertRows) and experts is None:
+            experts = piece
+        elif isinstance(piece, PartialSums) and piece.dtype is None:
+            dense.append((piece.data, piece.parts, piece.rows * piece.hidden))
+        elif piece is not None:
+            piece = materialize(piece)
+            _need(piece, torch.float32, "delta")
+            dense.append((piece, 1, 0))
+    dense += [(None, 0, 0)] * (2 - len(dense))
+    rows_ptr = pos = ids = wts = None
+    top_k, eparts, estride = 0, 1, 0
+    if experts is not None:
+        rows_ptr, pos, ids, wts, top_k = experts.rows, experts.pos_of_pair, experts.ids, experts.wts, experts.ids.shape[1]
+        if experts.parts > 1:
+            eparts, estride = experts.parts, experts.rows.shape[1] * experts.rows.shape[2]
+    r = route or {}
+    if route:
+        _need(r["weight"], torch.float32, "router weight"); _need(r["ids"], torch.int32, "ids"); _need(r["wts"], torch.float32, "wts")
+    (d1, n1, s1), (d2, n2, s2) = dense
+    check(core().tl_add_rmsnorm_pair(
+        ptr(residual), ptr(d1), n1, s1, ptr(d2), n2, s2, ptr(rows_ptr), eparts, estride, ptr(pos), ptr(ids), ptr(wts), top_k,
+        ptr(weight), ptr(out), ptr(weight2), ptr(out2), ptr(gather), out.shape[0], residual.shape[-1], float(eps),
+        dtype_code(out.dtype), ptr(r.get("weight")), ptr(r.get("bias")), r["weight"].shape[0] if route else 0, int(r.get("k", 0)),
+        route_flags(r.get("normalize", 0), r.get("scoring", "sigmoid"), r.get("groups")), float(r.get("floor", 0.0)),
+        float(r.get("scale", 1.0)), ptr(r.get("ids")), ptr(r.get("wts")), stream()), "add_rmsnorm_pair")
+    return out
+
+
+def normed_sum(a, b, weight_a: torch.Tensor, weight_b: torch.Tensor, eps: float, scale: float, out: torch.Tensor) -> torch.Tensor:
+    """out = scale * (weight_a * a / rms(a) + weight_b * b / rms(b)) row by row in 32-bit; `a`, `b` float32 tensors or `PartialSums`."""
+    _need(out, torch.float32, "out"); _need(weight_a, torch.float32, "norm weight"); _need(weight_b, torch.float32, "norm weight")
+    rows, hidden = out.shape
+    pieces = []
+    for x in (a, b):
+        if isinstance(x, PartialSums) and x.dtype is None:
+            pieces.append((x.data, x.parts))
+        else:
+            x = materialize(x)
+            _need(x, torch.float32, "branch")
+            pieces.append((x, 1))
+    check(core().tl_normed_sum(ptr(pieces[0][0]), pieces[0][1], ptr(pieces[1][0]), pieces[1][1], rows * hidden, ptr(weight_a),
+                               ptr(weight_b), float(eps), float(scale), ptr(out), rows, hidden, stream()), "normed_sum")
     return out
 
 
@@ -602,10 +690,10 @@ def gemm_simt(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None, out: 
 def gemm_simt_grouped(a: torch.Tensor, a_gather: torch.Tensor | None, a_div: int, w: torch.Tensor, out: torch.Tensor,
                       plan: "MoePlan", swiglu: bool | int) -> torch.Tensor:
     """Per sorted row i of the plan: out[i] = A[row(i)] @ w[expert(i)]^T, with w [E, N(*2 when swiglu), K]. `swiglu`:
-    False for a plain product, True or a code of ACTIVATIONS for act(gate rows) * (up rows)."""
+    False for a plain product, True or a code of ACTIVATIONS for act(gate rows) * (up rows), a negated code for act(plain product)."""
     _need(a, w.dtype, "a"); _need(w, None, "w"); _need(out, None, "out")
     E, n_rows_w, K = w.shape
-    N = n_rows_w // 2 if swiglu else n_rows_w
+    N = n_rows_w // 2 if int(swiglu) > 0 else n_rows_w
     check(core().tl_gemm_simt_grouped(ptr(a), a.stride(0), ptr(a_gather), a_div, ptr(w), w.stride(1), w.stride(0),
                                       ptr(out), out.stride(0), plan.pairs, N, K, ptr(plan.tile_group),
                                       ptr(plan.tile_row0), ptr(plan.tile_rows), ptr(plan.n_tiles), plan.max_tiles,
@@ -734,12 +822,15 @@ def attention_join(scratch, positions, window, out, n_spans: int, span_keys: int
 
 def qkv_rotate_store(qkv, q_col: int, k_col: int, v_col: int, inv_freq, rot: int, inv_freq_v, positions, req_of_row, table,
                      page_size: int, q_out, k_cache, v_cache, num_heads: int, num_kv_heads: int, head_dim: int, value_dim: int,
-                     status, rot_magnitude: float = 1.0, v_other=None, v_blend=None) -> None:
+                     status, rot_magnitude: float = 1.0, v_other=None, v_blend=None, q_weight=None, k_weight=None,
+                     norm_eps: float = 0.0, neighbours: bool = False) -> None:
     """From the rows of one fused product (`q_col`, `k_col`, `v_col`: where each part begins in a row; `k_col` < 0: the rows
     hold queries only): rotary over the first `rot` entries of every q and k head (halves layout; `inv_freq` None: none), its
     sines and cosines times `rot_magnitude`; the values turned over all their entries by `inv_freq_v` (None: as projected), or
     blended with the same rows of `v_other` (a view [rows, kv heads * value_dim] of the compute dtype, unit inner stride):
-    (1 - l) v + l v_other with l = `v_blend` (float32, one number on the device); q to `q_out`, k and v into their pages."""
+    (1 - l) v + l v_other with l = `v_blend` (float32, one number on the device); q to `q_out`, k and v into their pages. With
+    `q_weight` and `k_weight` (float32 [head_dim]) every q and k head is first divided by its root mean square and multiplied by
+    the weight; with `neighbours` entries 2i and 2i + 1 are the pairs that turn."""
     _need(qkv, None, "qkv"); _need(q_out, qkv.dtype, "q")
     if v_other is not None and (v_other.dtype != qkv.dtype or v_other.stride(1) != 1 or
                                 v_other.shape != (qkv.shape[0], num_kv_heads * value_dim)):
@@ -750,16 +841,20 @@ def qkv_rotate_store(qkv, q_col: int, k_col: int, v_col: int, inv_freq, rot: int
                                      k_cache.shape[0] if k_cache is not None else 0, ptr(q_out), ptr(k_cache), ptr(v_cache),
                                      qkv.shape[0], num_heads, num_kv_heads, head_dim, value_dim, dtype_code(qkv.dtype),
                                      ptr(status), float(rot_magnitude), ptr(v_other),
-                                     v_other.stride(0) if v_other is not None else 0, ptr(v_blend), stream()),
+                                     v_other.stride(0) if v_other is not None else 0, ptr(v_blend), ptr(q_weight), ptr(k_weight),
+                                     float(norm_eps), int(neighbours), stream()),
           "qkv_rotate_store")
 
 
 def attention_flex(q, k_cache, v_cache, table, page_size: int, req_of_row, positions, scale: float, softcap, window,
-                   keep_first: int, inv_freq_out, gate, ld_gate: int, out_scale: float, out, status) -> torch.Tensor:
+                   keep_first: int, inv_freq_out, gate, ld_gate: int, out_scale: float, out, status, chunk: int | None = None,
+                   sinks: torch.Tensor | None = None, gate_heads: bool = False) -> torch.Tensor:
     """Attention of every row over its request's pages: capped scores (`softcap` None: none), a window that also keeps the
     first `keep_first` tokens (`window` None: all keys), the output turned back by `inv_freq_out` (None: not), times
     sigmoid(`gate`) entry by entry (a tensor of the compute dtype beginning at the first logit, rows `ld_gate` apart), times
-    `out_scale`. `out` [rows, heads * value_dim] may be a column slice of a wider tensor."""
+    `out_scale`. `out` [rows, heads * value_dim] may be a column slice of a wider tensor. With `chunk` a row sees the keys of its own
+    chunk of positions only; `sinks` (float32 [heads]): exp(sink) is in a head's denominator; `gate_heads`: the gate has one logit a
+    head."""
     _need(q, k_cache.dtype, "q")
     rows, Hq, D = q.shape
     Hk, VD = k_cache.shape[1], v_cache.shape[3]
@@ -769,7 +864,7 @@ def attention_flex(q, k_cache, v_cache, table, page_size: int, req_of_row, posit
                                    k_cache.shape[0], ptr(req_of_row), ptr(positions), float(scale), float(softcap or 0.0),
                                    int(window or 0), int(keep_first or 0), ptr(inv_freq_out), ptr(gate), int(ld_gate),
                                    float(out_scale), ptr(out), out.stride(0), rows, Hq, Hk, D, VD, dtype_code(q.dtype),
-                                   ptr(status), stream()), "attention_flex")
+                                   ptr(status), int(chunk or 0), ptr(sinks), int(gate_heads), stream()), "attention_flex")
     return out
 
 
@@ -803,6 +898,62 @@ def recurrence_scan(proj, q_col: int, k_col: int, v_col: int, state, state_slot,
                                     ptr(scratch), rows, sm_count(), rule, float(q_scale), stream()), "recurrence_scan",
           kernels=2 if scratch is not None else 1)
     return y
+
+
+def gated_delta_scan(proj, cols: dict, taps, conv_cols: int, slots, state_offset: int, step, y, heads: int, groups: int, key_dim: int,
+                     value_dim: int, a_log, dt_bias, *, unit_eps: float, q_scale: float, decay_logits=None, write_state: bool = True
+                     ) -> torch.Tensor:
+    """The gated delta rule (csrc/recurrence_write.cu) over the rows of `step`. `proj` float32 rows with q, k (`groups` heads), v and
+    the write strengths' logits at `cols` ("q", "k", "v", "b"), whose first `conv_cols` columns pass the convolution `taps` (float32
+    [conv_cols, K]); the decays' logits one a head at cols["a"], or one a head and key channel in `decay_logits` (float32 [rows,
+    heads * key_dim]). `slots` float32 [slots, floats]: a slot's convolution inputs at its beginning, its state [heads, values, keys]
+    `state_offset` floats behind. `y` float32 [rows, heads * value_dim]."""
+    _need(proj, torch.float32, "projections"); _need(slots, torch.float32, "slots"); _need(y, torch.float32, "y"); _need(taps, torch.float32, "taps")
+    rows = proj.shape[0]
+    rule = 4 if decay_logits is None else 3
+    if decay_logits is not None and (decay_logits.dtype != torch.float32 or decay_logits.stride(1) != 1):
+        raise KernelError("gated delta rule: float32 decay logits with unit stride")
+    scratch = None
+    if step.max_rows_per_request > RECURRENCE_STAGED_ROWS:
+        scratch = torch.empty(core().tl_write_scan_scratch_floats(rows, heads, key_dim, value_dim, rule), dtype=torch.float32,
+                              device=proj.device)
+    check(core().tl_gated_delta_scan(
+        ptr(proj), proj.stride(0), cols["q"], cols["k"], cols["v"], cols["b"], cols["a"] if decay_logits is None else -1,
+        ptr(decay_logits), decay_logits.stride(0) if decay_logits is not None else 0, ptr(a_log), ptr(dt_bias), float(unit_eps),
+        float(q_scale), ptr(taps), taps.shape[1], int(conv_cols), ptr(slots), slots.stride(0), int(state_offset), ptr(step.state_slot),
+        ptr(step.row_start), ptr(step.req_of_row), step.n_requests, ptr(y), heads, groups, key_dim, value_dim, int(write_state),
+        ptr(scratch), rows, sm_count(), stream()), "gated_delta_scan", kernels=2 if scratch is not None else 1)
+    return y
+
+
+def matrix_memory_scan(proj, cols: dict, i_bias, f_bias, cap: float, slots, state_offset: int, step, y, maxima, heads: int,
+                       key_dim: int, value_dim: int, *, q_scale: float, write_state: bool = True) -> torch.Tensor:
+    """The gated matrix memory (csrc/recurrence_write.cu): `proj` float32 rows with q, k, v and the two gates' logits at `cols` ("q",
+    "k", "v", "i", "f"); a slot's running maxima at its beginning and its state [heads, values + 1, keys] `state_offset` floats
+    behind. `y` float32 [rows, heads * (value_dim + 1)]: a head's outputs and, behind them, n . q; `maxima` float32 [rows, heads]."""
+    _need(proj, torch.float32, "projections"); _need(slots, torch.float32, "slots"); _need(y, torch.float32, "y")
+    rows = proj.shape[0]
+    factors = torch.empty(rows, heads, 2, dtype=torch.float32, device=proj.device)
+    scratch = None
+    if step.max_rows_per_request > RECURRENCE_STAGED_ROWS:
+        scratch = torch.empty(core().tl_write_scan_scratch_floats(rows, heads, key_dim, value_dim + 1, 5), dtype=torch.float32,
+                              device=proj.device)
+    check(core().tl_matrix_memory_scan(
+        ptr(proj), proj.stride(0), cols["q"], cols["k"], cols["v"], cols["i"], cols["f"], ptr(i_bias), ptr(f_bias), float(cap),
+        float(q_scale), ptr(slots), slots.stride(0), int(state_offset), ptr(step.state_slot), ptr(step.row_start), step.n_requests,
+        ptr(y), ptr(maxima), ptr(factors), heads, key_dim, value_dim, int(write_state), ptr(scratch), rows, sm_count(), stream()),
+        "matrix_memory_scan", kernels=3 if scratch is not None else 2)
+    return y
+
+
+def memory_norm_gate(y, maxima, gate, weight, eps: float, floor: float, out, heads: int, value_dim: int) -> torch.Tensor:
+    """What follows `matrix_memory_scan`: a head's outputs over max(|n . q|, exp(-maximum)) + floor, brought to unit root mean square,
+    times `weight` [heads * value_dim], times sigmoid(gate); `gate` a float32 view [rows, >= heads * value_dim] of unit stride."""
+    if gate.dtype != torch.float32 or gate.stride(1) != 1 or out.stride(1) != 1:
+        raise KernelError("memory norm: a float32 gate and an output of unit stride")
+    check(core().tl_memory_norm_gate(ptr(y), ptr(maxima), ptr(gate), gate.stride(0), ptr(weight), float(eps), float(floor), ptr(out),
+                                     out.stride(0), y.shape[0], heads, value_dim, dtype_code(out.dtype), stream()), "memory_norm_gate")
+    return out
 
 
 def group_norm_gate(y, gate, ld_gate: int, weight, eps: float, groups: int, scale: float, out, gate_activation: str = "sigmoid"

@@ -127,7 +127,7 @@ def lib():
         l.tl_attention_flex_mma.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int,
                                             c_void_p, ctypes.c_float, ctypes.c_float, c_int, c_int, c_void_p, c_void_p, c_longlong,
                                             ctypes.c_float, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                            c_void_p, c_void_p]
+                                            c_void_p, c_int, c_void_p, c_int, c_void_p]
         l.tl_attention_flex_mma.restype = c_int
         l.tl_gemm_skinny_supported.argtypes = [c_int, c_int, c_int, c_longlong, c_longlong]
         l.tl_gemm_skinny_supported.restype = c_int
@@ -172,17 +172,20 @@ class TensorCore:
     def __init__(self, device, status: torch.Tensor):
         self.device, self.status = device, status
         self.sm_count = torch.cuda.get_device_properties(device).multi_processor_count
-        self._workspace = None
+        self.branch = 0             # which of several chains of products that keep partial sums for one norm is running
+        self._workspaces = {}
         self._pair_order = None
         self._pairs = None
         self._outgrown = []
 
     def workspace(self, floats: int) -> torch.Tensor:
-        if self._workspace is None or self._workspace.numel() < floats:
-            if self._workspace is not None:
-                self._outgrown.append(self._workspace)      # a captured decode graph may still write to the smaller one
-            self._workspace = torch.empty(max(floats, 1 << 20), dtype=torch.float32, device=self.device)
-        return self._workspace
+        """The running branch's buffer for partial sums: what one product left there is gone with the next one's of that branch."""
+        buf = self._workspaces.get(self.branch)
+        if buf is None or buf.numel() < floats:
+            if buf is not None:
+                self._outgrown.append(buf)      # a captured decode graph may still write to the smaller one
+            buf = self._workspaces[self.branch] = torch.empty(max(floats, 1 << 20), dtype=torch.float32, device=self.device)
+        return buf
 
     # ---- x @ w^T (+ bias) ----
     def gemm(self, x, w2d, bias, out, *, rows_per_group=0, plan=None, swiglu=False, swap=None, bn=None, n_out=None,
@@ -404,7 +407,7 @@ class TensorCore:
         one, whose CTAs of 128 outputs are few and each wait for a TMA ring to fill. The plan is built in tiles of 8 rows,
         which is what a CTA of that product takes."""
         E, I2, H = part.w_gate_up.shape
-        inter, (R, k) = I2 // 2, ids.shape
+        inter, (R, k) = part.inter, ids.shape
         P = R * k
         act = torch.empty(P, inter, dtype=x.dtype, device=x.device)
         y = torch.empty(P, H, dtype=torch.float32, device=x.device)
@@ -444,8 +447,8 @@ class TensorCore:
     def experts(self, part, x, ids, wts, plan=None):
         """The routed experts of `part` on rows x: an `ops.ExpertRows` (to be weighed and added per row), or None
         when the kernels do not take the shapes. `plan`: the routing plan when something built it already."""
-        E, I2, H = part.w_gate_up.shape
-        inter = I2 // 2
+        E, I2, H = part.w_gate_up.shape          # (without a gate: the up rows alone, and `part.act` is negative)
+        inter = part.inter
         if not usable(x, part.w_gate_up.view(E * I2, H)) or inter % 8 or not part.w_down.is_contiguous():
             return None
         R, k = ids.shape
@@ -574,7 +577,7 @@ def _attention_flex(self, part, q, cache, table, step, gate, ld_gate: int, out_s
             cache.k.shape[0], tiles.data_ptr(), tiles.shape[0], int(most), step.positions.data_ptr(), float(part.scale),
             float(part.softcap or 0.0), int(part.window or 0), int(part.keep_first or 0), ops.ptr(part.inv_freq_v), ops.ptr(gate),
             int(ld_gate), float(out_scale), out.data_ptr(), out.stride(0), R, Hq, Hk, D, VD, int(step.max_context), ops.sm_count(),
-            self.status.data_ptr(), ops.stream())
+            self.status.data_ptr(), int(part.chunk or 0), ops.ptr(part.sinks), int(part.gate_heads), ops.stream())
         _check(code, "attention_flex_mma")
     return True
 

@@ -26,8 +26,11 @@ Options, each a parameter of the spec so that another design can name its own co
               leaves its values as projected (`blend` None there); a later layer with the same `key` caches and attends over
               (1 - l) v + l v_first, l the one number stored as `<prefix><blend>`, v_first the first layer's values of the same
               row. Both must have the same number of KV heads and value size.
+  `chunk` n: a row sees the keys j <= i of its own chunk of n positions (counted from position 0) instead of a window;
+  `sinks`: the name of a vector [Hq]: exp(sink_h) is in head h's softmax denominator, without a key or a value, unscaled.
 A position encoding whose sines and cosines carry a factor (`magnitude`) passes it to the q/k kernel.
-Any of these takes the mixer to the kernels of csrc/attention_flex.cu, which have all of them as arguments.
+Any of these from `value_dim` on, or interleaved rotary pairs, takes the mixer to the kernels of csrc/attention_flex.cu, which have
+all of them as arguments, and q/k norms with weights and a gate a head besides.
 
 Every size (heads, KV heads, head size), the scale, the window and the names of its tensors are
 parameters. The q, k and v matrices are fused into one product at bind time, as the reference's loader
@@ -57,11 +60,11 @@ class AttentionMixer(Part):
         self.head_dim = int(spec["head_dim"])
         if self.num_heads % self.num_kv_heads:
             raise ValueError(f"{self.num_heads} query heads are not a multiple of {self.num_kv_heads} KV heads")
-        if spec.get("head_mix") or spec.get("gate"):
+        flexible = ("softcap", "keep_first", "value_rotation", "entry_gate", "borrows_keys", "bias", "value_carry", "chunk", "sinks")
+        if spec.get("head_mix") or (spec.get("gate") and not any(spec.get(k) for k in flexible)):
             if not 1 <= self.head_dim <= 256:       # the head-mixing kernels take any head size the q/k kernel does
                 raise ValueError(f"head size {self.head_dim}: 1 to 256 are implemented")
-        elif any(spec.get(k) for k in ("softcap", "keep_first", "value_rotation", "entry_gate", "borrows_keys", "bias",
-                                       "value_carry")) or \
+        elif any(spec.get(k) for k in flexible) or spec["position"].kind == "rope_pairs" or \
                 int(spec.get("value_dim") or self.head_dim) != self.head_dim:
             if not (1 <= self.head_dim <= 256 and 1 <= int(spec.get("value_dim") or self.head_dim) <= 256):
                 raise ValueError(f"head sizes {self.head_dim} and {spec.get('value_dim')}: 1 to 256 are implemented")
@@ -97,18 +100,31 @@ class AttentionMixer(Part):
         self.carry_key = str(carry["key"]) if carry else None
         self.carry_blend_name = prefix + carry["blend"] if carry and carry.get("blend") else None
         self.bias_suffix = str(spec.get("bias_suffix", ".b"))
+        self.chunk = int(spec["chunk"]) if spec.get("chunk") else None
+        self.sinks_name = prefix + spec["sinks"] if spec.get("sinks") else None
+        self.pairs = hasattr(self.position, "fused_rotary_pairs")
         self.flex = bool(self.value_dim != self.head_dim or self.softcap or self.keep_first or self.value_rotation
-                         or self.entry_gate_name or self.borrows_keys or self.bias or carry
+                         or self.entry_gate_name or self.borrows_keys or self.bias or carry or self.chunk or self.sinks_name
+                         or self.pairs
                          or getattr(self.position, "magnitude", 1.0) != 1.0)
         if self.flex:
-            if self.head_mix_name or self.gate_name or self.q_norm or self.values != "projected":
-                raise ValueError("capped scores, kept first tokens, turned values, an entry-wise gate and borrowed keys do "
-                                 "not combine with mixed heads, a gate a head, q/k norms or values that are the keys")
+            if self.head_mix_name or self.values != "projected" or (self.q_norm and qk.kind != "rmsnorm") or \
+                    (self.q_norm and self.borrows_keys) or (self.gate_name and self.entry_gate_name):
+                raise ValueError("capped scores, kept first tokens, chunks, sinks, turned values, an entry-wise gate and borrowed "
+                                 "keys do not combine with mixed heads, weightless q/k norms or values that are the keys, "
+                                 "borrowed keys not with q/k norms, an entry-wise gate not with one a head")
+            if self.chunk and (self.window or self.keep_first):
+                raise ValueError("chunks of positions do not combine with a window")
             if self.value_rotation and self.value_dim % 2:
                 raise ValueError(f"values of odd size {self.value_dim} cannot be turned in pairs")
             if carry and (self.value_rotation or self.borrows_keys):
                 raise ValueError("carried values are neither turned nor borrowed")
-        self.inv_freq_v = self.b_qkv = self.b_out = self.carry_blend = None
+        self.inv_freq_v = self.b_qkv = self.b_out = self.carry_blend = self.sinks = None
+
+    @property
+    def gate_heads(self) -> bool:
+        """The gate has one logit a head (not one an entry)."""
+        return bool(self.gate_name)
 
     @property
     def out_dim(self) -> int:
@@ -131,6 +147,12 @@ class AttentionMixer(Part):
                         TensorSpec(self.n["v"] + sfx, (self.num_kv_heads * self.value_dim, H))]
             if self.entry_gate_name:
                 out.append(TensorSpec(self.entry_gate_name + sfx, (self.out_dim, H)))
+            if self.gate_name:
+                out.append(TensorSpec(self.gate_name, (self.num_heads, H)))
+            if self.sinks_name:
+                out.append(TensorSpec(self.sinks_name, (self.num_heads,), "vector", "bias"))
+            if self.q_norm:
+                out += self.q_norm.weight_specs() + self.k_norm.weight_specs()
             out.append(TensorSpec(self.n["out"] + sfx, (H, self.out_dim)))
             if self.bias:
                 sizes = {"q": self.q_dim, "k": self.kv_dim, "v": self.num_kv_heads * self.value_dim, "out": H}
@@ -161,6 +183,13 @@ class AttentionMixer(Part):
             mats = [(x, runtime.matrix(read(self.n[x] + sfx))) for x in parts]
             if self.entry_gate_name:
                 mats.append(("gate", runtime.matrix(read(self.entry_gate_name + sfx))))
+            if self.gate_name:
+                mats.append(("gate", runtime.matrix(read(self.gate_name))))
+            if self.sinks_name:
+                self.sinks = runtime.vector(read(self.sinks_name))
+            if self.q_norm:
+                self.q_norm.bind(read, runtime)
+                self.k_norm.bind(read, runtime)
             rows, self.col, at = [], {}, 0
             for name, m in mats:
                 self.col[name] = at
@@ -204,7 +233,7 @@ class AttentionMixer(Part):
         if self.flex:
             return PagedNeed(self.num_kv_heads, self.head_dim, self.cache_window,
                              value_dim=self.value_dim if self.value_dim != self.head_dim else None,
-                             keep_first=self.cache_keep_first if self.cache_window else 0)
+                             keep_first=self.cache_keep_first if self.cache_window else 0, chunk=self.chunk)
         return PagedNeed(self.num_kv_heads, self.head_dim, self.window)
 
     def forward_inner(self, x, step, cache, writes_cache: bool, out: torch.Tensor, out_scale: float = 1.0) -> torch.Tensor:
@@ -218,7 +247,9 @@ class AttentionMixer(Part):
         qkv = linear(self.runtime, x, self.w_qkv, self.b_qkv)
         q = torch.empty(R, Hq, D, dtype=dt, device=dev)
         table = step.block_tables[cache.group]
-        inv_freq, rot = self.position.fused_rotary()
+        inv_freq, rot = self.position.fused_rotary_pairs() if self.pairs else self.position.fused_rotary()
+        if not rot:
+            inv_freq = None
         own = writes_cache and not self.borrows_keys
         v_other = None
         if self.carry_key is not None:
@@ -232,15 +263,17 @@ class AttentionMixer(Part):
         ops.qkv_rotate_store(qkv, self.col["q"], self.col["k"] if own else -1, self.col["v"] if own else -1, inv_freq, rot,
                              self.inv_freq_v, step.positions, step.req_of_row, table, cache.page_size, q,
                              cache.k if own else None, cache.v if own else None, Hq, Hk, D, VD, status,
-                             float(getattr(self.position, "magnitude", 1.0)), v_other, self.carry_blend)
-        gate = qkv[:, self.col["gate"]:] if self.entry_gate_name else None
+                             float(getattr(self.position, "magnitude", 1.0)), v_other, self.carry_blend,
+                             self.q_norm.weight if self.q_norm else None, self.k_norm.weight if self.q_norm else None,
+                             self.q_norm.eps if self.q_norm else 0.0, self.pairs)
+        gate = qkv[:, self.col["gate"]:] if "gate" in self.col else None
         fast = self.runtime.attention_kernels
         if fast is not None and hasattr(fast, "attention_flex") and fast.attention_flex(self, q, cache, table, step, gate,
                                                                                        qkv.stride(0), out_scale, out):
             return out
         return ops.attention_flex(q, cache.k, cache.v, table, cache.page_size, step.req_of_row, step.positions, self.scale,
                                   self.softcap, self.window, self.keep_first, self.inv_freq_v, gate, qkv.stride(0), out_scale,
-                                  out, status)
+                                  out, status, self.chunk, self.sinks, self.gate_heads)
 
     def forward(self, x, step, cache, writes_cache: bool = True):
         if self.flex:

@@ -31,7 +31,7 @@ Interfaces (duck-typed; the base classes below document them and hold the shared
                   an `ops.StreamUpdate`, which the next norm's kernel takes into the streams.
 
 A branch output is what a mixer or feed-forward adds to the residual stream: a float32 tensor [R, hidden], or one of
-the deferred forms of `kernels.ops` (`PartialSums`, `ExpertRows`) that the next norm kernel adds itself;
+the deferred forms of `kernels.ops` (`PartialSums`, `ExpertRows`, a `BranchSum` of two) that the next norm kernel adds itself;
 `kernels.ops.materialize` turns any of them into a tensor.
 
 `step` is the `StepContext` of the running batch: rows of several requests flattened, with each row's
@@ -49,6 +49,7 @@ appends (its prefix, the chosen expert ids) under "routes"); a traced step alway
 
 from __future__ import annotations
 
+from contextlib import contextmanager
 from dataclasses import dataclass, field
 from typing import Any, Callable
 
@@ -101,10 +102,27 @@ class Runtime:
         if self.status is None and self.device.type == "cuda":
             self.status = torch.zeros(1, dtype=torch.int32, device=self.device)
 
+    @contextmanager
+    def branch(self, index: int):
+        """Inside, parts belong to branch `index` of several whose results one later kernel adds: every branch keeps its partial
+        sums and its scratch in buffers of its own, so that one branch's are not overwritten by another's products. Branches nest
+        (the indices of nested branches add up); outside of any the index is 0."""
+        before = self.__dict__.get("_branch", 0)
+        self.__dict__["_branch"] = before + index
+        if self.tensorcore is not None:
+            self.tensorcore.branch = before + index
+        try:
+            yield
+        finally:
+            self.__dict__["_branch"] = before
+            if self.tensorcore is not None:
+                self.tensorcore.branch = before
+
     def scratch(self, name: str, numel: int, dtype: torch.dtype = torch.float32) -> torch.Tensor:
         """A kept device buffer of at least `numel` elements for a kernel's intermediate results. Kernels on one
         stream run in order, so parts that run one after another may share a name."""
         pool = self.__dict__.setdefault("_scratch", {})
+        name = f"{name}/{self.__dict__.get('_branch', 0)}"
         buf = pool.get((name, dtype))
         if buf is None or buf.numel() < numel:
             if buf is not None:
@@ -130,6 +148,12 @@ class PagedNeed:
     values: bool = True         # False: nothing is stored beside the keys (the site's `v` is its `k`)
     value_dim: int | None = None    # size of a value a head where it differs from a key's (None: head_dim)
     keep_first: int = 0         # with a window: positions below this stay readable for good, so their pages are kept
+    chunk: int | None = None    # a position only reads its own chunk of this many, counted from 0, so the chunks before go back
+
+    @property
+    def reach(self) -> int | None:
+        """The most positions a row reads (None: all before it), without the kept first ones."""
+        return self.window if self.window is not None else self.chunk
 
 
 @dataclass(frozen=True)

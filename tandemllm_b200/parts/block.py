@@ -15,6 +15,14 @@ The norm behind a branch, the residual add and the norm in front of the next sub
 sublayer is in the same layer (`add_normed(..., then=next norm)`); a layer hands nothing pending to the next one, so
 that whatever a run order adds to the stream between two layers meets a complete residual.
 
+`parallel_residual` lets the mixer and the feed-forward read two norms of the same residual:
+
+    h = h + (mixer(norm_m(h)) + feed_forward(norm_f(h)))
+
+Both norms are one kernel behind the adds of what the layer before left (`add_two_norms`), with the router of a routed
+feed-forward inside; what the layer leaves is an `ops.BranchSum`, which the next norm's kernel adds. The feed-forward runs as
+a branch of its own (`Runtime.branch`): its partial sums and the mixer's wait side by side.
+
 `hyper_connections` carries several residual streams x_1 .. x_S [S, rows, hidden] instead of one. Sublayer q of a layer
 (1: mixer, 2: feed-forward) has three small tensors, `<prefix>hc<q>.in` [S], `.out` [S] and `.mix` [S, S] (indexed [from, to]):
 
@@ -64,6 +72,19 @@ class SandwichNormResidual:
         else:
             layer.feed_forward_post_norm.add_normed(residual, out)
         return None
+
+
+@register_part("arrangement", "parallel_residual")
+class ParallelResidual:
+    def run(self, layer: "Layer", residual, pending, step, cache, writes_cache: bool = True):
+        ff = layer.feed_forward
+        if getattr(ff, "absent", False):
+            return layer.mixer.forward(layer.mixer_norm.add_norm(residual, pending), step, cache, writes_cache=writes_cache)
+        route = ff.router_args(residual.shape[0], residual.device) if hasattr(ff, "router_args") else None
+        n, nf = layer.mixer_norm.add_two_norms(residual, pending, layer.feed_forward_norm, route)
+        with ff.runtime.branch(1):
+            out = ff.forward(nf, step, routing=(route["ids"], route["wts"])) if route is not None else ff.forward(nf, step)
+        return ops.BranchSum(layer.mixer.forward(n, step, cache, writes_cache=writes_cache), out)
 
 
 class _Reading:

@@ -6,6 +6,9 @@
            times scale; out = sum over the chosen experts in ascending expert id of w * expert(n)
                                                                          ref.py:185-214
 
+With `gated: False` an expert has no gate matrix: expert(n) = down( act(up n) ), the activation in the up product's epilogue.
+With the scoring `chosen_softmax` the bias is part of the logits, and the weights are the softmax over the chosen experts' logits.
+
 The gate's activation (`activation`: silu, gelu, relu2, identity) and the router's scoring function (`scoring`:
 sigmoid, or softmax over all experts) are parameters of the parts' specs, passed to the kernels as codes; LFM2 uses
 silu and sigmoid, and another architecture's gated or routed feed-forward reuses the same fused kernels by naming its own.
@@ -146,6 +149,11 @@ class SigmoidTopKExperts(Part):
         ops.route_flags(self.normalize, self.scoring, self.groups)      # an unknown scoring function is refused here
         self.act = ops.activation_code(spec.get("activation", "silu"))
         self.gate_constants = gate_constants_of(spec)
+        self.gated = bool(spec.get("gated", True))
+        if not self.gated:
+            if self.act > ops.ACTIVATIONS["identity"]:
+                raise ValueError(f"ungated experts with the activation {spec.get('activation')!r}: silu, gelu, relu2 or identity")
+            self.act = -self.act            # how the grouped products are asked for the ungated form
         self.suffix = str(spec.get("weight_suffix", ".weight"))
         self.sep = str(spec.get("expert_separator", "."))       # between the experts' common name and an expert's number
         if not 0 < self.top_k <= self.num_experts:
@@ -160,7 +168,7 @@ class SigmoidTopKExperts(Part):
         self.load = None            # see `count_into`
 
     def _stacked(self, present) -> bool:
-        return present is not None and (self.base + ".gate_up_proj") in present
+        return self.gated and present is not None and (self.base + ".gate_up_proj") in present
 
     def weight_specs(self, present=None):
         H, I, E = self.hidden_size, self.inter, self.num_experts
@@ -172,8 +180,8 @@ class SigmoidTopKExperts(Part):
             out += [TensorSpec(self.base + ".gate_up_proj", (E, 2 * I, H)), TensorSpec(self.base + ".down_proj", (E, H, I))]
         else:
             for e in range(E):
-                out += [TensorSpec(self._expert(e, "gate"), (I, H)), TensorSpec(self._expert(e, "up"), (I, H)),
-                        TensorSpec(self._expert(e, "down"), (H, I))]
+                out += [TensorSpec(self._expert(e, "gate"), (I, H))] if self.gated else []
+                out += [TensorSpec(self._expert(e, "up"), (I, H)), TensorSpec(self._expert(e, "down"), (H, I))]
         return out
 
     def _expert(self, e: int, which: str) -> str:
@@ -189,11 +197,13 @@ class SigmoidTopKExperts(Part):
             self.w_gate_up = runtime.matrix(read(self.base + ".gate_up_proj"))
             self.w_down = runtime.matrix(read(self.base + ".down_proj"))
         else:
-            self.w_gate_up = torch.empty(E, 2 * I, H, dtype=runtime.dtype, device=runtime.device)
+            up_at = I if self.gated else 0          # (without a gate the up rows are all there is)
+            self.w_gate_up = torch.empty(E, up_at + I, H, dtype=runtime.dtype, device=runtime.device)
             self.w_down = torch.empty(E, H, I, dtype=runtime.dtype, device=runtime.device)
             for e in range(E):
-                self.w_gate_up[e, :I].copy_(read(self._expert(e, "gate")))
-                self.w_gate_up[e, I:].copy_(read(self._expert(e, "up")))
+                if self.gated:
+                    self.w_gate_up[e, :I].copy_(read(self._expert(e, "gate")))
+                self.w_gate_up[e, up_at:].copy_(read(self._expert(e, "up")))
                 self.w_down[e].copy_(read(self._expert(e, "down")))
 
     def expected_experts_read(self, rows: int) -> float:
@@ -206,7 +216,7 @@ class SigmoidTopKExperts(Part):
         of distinct experts `rows` rows choose)."""
         H, I, E = self.hidden_size, self.inter, self.num_experts
         n = self.expected_experts_read(rows) if experts_read is None else experts_read
-        return int(E * H * 4 + (E * 4 if self.use_bias else 0) + n * 3 * H * I * elem)
+        return int(E * H * 4 + (E * 4 if self.use_bias else 0) + n * (3 if self.gated else 2) * H * I * elem)
 
     def count_into(self, counts: torch.Tensor | None) -> None:
         """From now on every pass adds the pairs it routed to each expert to `counts` (an integer tensor [experts] on

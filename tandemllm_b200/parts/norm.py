@@ -60,6 +60,15 @@ class RMSNorm(Part):
         ops.add_rmsnorm(residual, delta, self.weight, self.eps, out, gather, out32, route)
         return out, out32
 
+    def add_two_norms(self, residual: torch.Tensor, delta, other: "RMSNorm", route: dict | None = None):
+        """residual += delta (a branch output or an `ops.BranchSum` of two); returns this norm's and `other`'s rows of the new
+        residual, both from one kernel (they divide by the same root mean square). `route`: a router run on `other`'s unrounded rows."""
+        if other.eps != self.eps:
+            raise ValueError(f"two norms of one row with different eps: {self.eps} and {other.eps}")
+        rows = residual.shape[0]
+        out, out2 = (torch.empty(rows, self.size, dtype=self.runtime.dtype, device=residual.device) for _ in range(2))
+        ops.add_rmsnorm_pair(residual, delta, self.weight, self.eps, out, other.weight, out2, None, route)
+        return out, out2
 
     def add_normed(self, residual: torch.Tensor, delta, gate: torch.Tensor | None = None, experts=None, then=None,
                    gather: torch.Tensor | None = None, n_out: int | None = None):
