@@ -234,8 +234,15 @@ def feed_forward(n, mlp, w, pre):
 MIXERS = {"channel_delta": mixer_channel_delta, "mlstm": mixer_mlstm, "parallel": mixer_parallel}
 
 
-def forward(config, weights, tokens, return_layers=False):
-    """Logits [T, vocab] of one whole sequence; with `return_layers` also the residual stream after every layer."""
+def choice_margin(z, top):
+    """[T]: how far the last chosen logit is above the first one left out."""
+    s = np.sort(z, axis=-1)[:, ::-1]
+    return s[:, top - 1] - s[:, top] if top < z.shape[1] else np.full(len(z), np.inf)
+
+
+def forward(config, weights, tokens, return_layers=False, margins=None):
+    """Logits [T, vocab] of one whole sequence; with `return_layers` also the residual stream after every layer. A list given as
+    `margins` receives every routed layer's `choice_margin`."""
     w = {k: np.asarray(v, dtype=np.float64) for k, v in weights.items()}
     eps = float(config["norm"]["eps"])
     x = w["embed"][np.asarray(tokens)]
@@ -247,7 +254,10 @@ def forward(config, weights, tokens, return_layers=False):
         pre = f"l{owner}."
         y = MIXERS[layer["type"]](plain_norm(x, w[pre + "norm1"], eps), layer["mixer"], w, pre + "mix.", eps)
         if layer.get("mlp"):
-            y = y + feed_forward(plain_norm(x, w[pre + "norm2"], eps), layer["mlp"], w, pre + "mlp.")
+            n = plain_norm(x, w[pre + "norm2"], eps)
+            y = y + feed_forward(n, layer["mlp"], w, pre + "mlp.")
+            if margins is not None and layer["mlp"]["kind"] == "moe":
+                margins.append(choice_margin(router_logits(n, w, pre + "mlp."), int(layer["mlp"]["router"]["top"])))
         x = x + y
         layers.append(x.copy())
     logits = plain_norm(x, w["final.norm"], eps) @ w["embed"].T
