@@ -22,6 +22,7 @@ requests at a context of 8192 tokens. A "step" is one decode step of the whole b
 `--design sebilorn` does the same for Sebilorn beside an LFM2 model of short-convolution and attention layers with dense
 feed-forwards.
 `--design niralix` does the same for Niralix beside an LFM2 MoE model of short-convolution and attention layers.
+`--design gifopel` does the same for Gifopel beside a Sebilorn model (matrix states and attention, dense) and an LFM2 MoE model.
 `--design sifupel` measures the Sifupel design beside the closest existing model (an LFM2 configuration of attention layers
 and dense feed-forwards only) at a few equal layer sizes: prefill and decode throughput, and every launch summed by kernel
 family with its fraction of the measured peak (its own line; the default workload and line are untouched).
@@ -380,7 +381,9 @@ class LaunchTimer:
                 "tl_group_norm_gate": "norm in parts + gate",
                 "tl_qkv_rotate_store": "rotary (+ turned values) + cache write", "tl_attention_flex": "attention",
                 "tl_attention_flex_mma": "attention", "tl_add_layernorm": "residual add + layer norm",
-                "tl_softcap": "logit cap"}.get(name, name)
+                "tl_softcap": "logit cap", "tl_add_rmsnorm_pair": "residual add + norm (+ router, + deferred sums)",
+                "tl_normed_sum": "two branches normed and averaged", "tl_gated_delta_scan": "gated delta rule (+ convolutions)",
+                "tl_matrix_memory_scan": "gated matrix memory", "tl_memory_norm_gate": "norm in parts + gate"}.get(name, name)
 
     def __enter__(self):
         torch = self.torch
@@ -1096,6 +1099,175 @@ def niralix_compare(a) -> int:
     return 0
 
 
+GIFOPEL_SIZES = {
+    "1k": dict(width=1024, layers=8, vocab=32768, heads=16, kv=4, dim=64, vdim=64, chunk=512, ff=2816, experts=16, top=4, expert_ff=704,
+               s_heads=16, s_kv=8, s_dim=64, s_vdim=64, context=1024),
+    "2k": dict(width=2048, layers=12, vocab=65536, heads=16, kv=4, dim=128, vdim=128, chunk=1024, ff=5632, experts=32, top=4,
+               expert_ff=1408, s_heads=16, s_kv=8, s_dim=128, s_vdim=128, context=2048),
+}
+
+
+def time_design(a, cfg, context: int) -> dict:
+    """A model with random weights from the typed configuration `cfg`: a prompt of `--prefill-tokens` tokens and decode steps of
+    `--batch` requests at `context` random cached positions (device-timed, medians of three; decode from CUDA graphs where the
+    engine takes them), and one prefill and one eager decode step with every launch timed and summed by kernel family."""
+    import torch
+
+    from tandemllm_b200.engine import Engine, EngineArgs, StepEntry
+    from tandemllm_b200.kernels import ops
+    from tandemllm_b200.sampling import SamplingParams
+    tokens, batch = a.prefill_tokens, a.batch
+    engine = Engine.from_config(cfg, seed=0, args=EngineArgs(
+        dtype=a.dtype, max_len=max(context, tokens) + 4 * a.steps + 64, parallel=batch, block_size=16,
+        max_batched_tokens=max(tokens, batch), chunk_size=tokens, graph=a.graph == "on"))
+    V = engine.model.vocab_size
+    for sc in engine.cache.site_cache:
+        for c in (sc if isinstance(sc, tuple) else (sc,)):
+            if getattr(c, "k", None) is not None:
+                c.k.normal_(0, 0.5)
+                if c.v is not None and c.v is not c.k:
+                    c.v.normal_(0, 0.5)
+    g = torch.Generator().manual_seed(1)
+    fn = engine.step_function
+
+    def prefill_once():
+        engine.admit("prefill")
+        prompt = torch.randint(0, V, (tokens,), generator=g).tolist()
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        engine.step([StepEntry("prefill", prompt, [tokens - 1])])
+        e1.record()
+        torch.cuda.synchronize()
+        engine.release("prefill")
+        return e0.elapsed_time(e1)
+    prefill_once()
+    pre_ms = statistics.median(prefill_once() for _ in range(5))
+    timer = LaunchTimer()
+    with timer:
+        prefill_once()
+        pre_table = timer.table()
+    greedy = SamplingParams(temperature=0.0, max_tokens=1 << 30, ignore_eos=True)
+    reqs = [start_with_context(engine, torch.randint(0, V, (context,), generator=g).tolist(), SamplingParams(**vars(greedy)))
+            for _ in range(batch)]
+    fn.check_status = False
+    toks = torch.randint(0, V, (3 * a.steps + a.warmup + 4, batch), generator=g).tolist()
+    picked = torch.empty(batch, dtype=torch.int32, device=engine.device)
+
+    def one(i):
+        ops.argmax(fn.run([StepEntry(r.request_id, [toks[i][j]], [0]) for j, r in enumerate(reqs)]), picked)
+    for i in range(a.warmup):
+        one(i)
+    torch.cuda.synchronize()
+    regions = []
+    for rep in range(3):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        for i in range(a.warmup + rep * a.steps, a.warmup + (rep + 1) * a.steps):
+            one(i)
+        e1.record()
+        torch.cuda.synchronize()
+        regions.append(e0.elapsed_time(e1) / a.steps)
+    dec_ms = statistics.median(regions)
+    fn.use_graphs = False
+    one(3 * a.steps + a.warmup)
+    with timer:
+        one(3 * a.steps + a.warmup + 1)
+        dec_table = timer.table()
+    fn.raise_on_fault()
+    for t in (pre_table, dec_table):
+        for r in t.values():
+            r["ms"] = round(r["ms"], 4)
+    nbytes = engine.model.decode_bytes(batch)["total"]
+    entry = {"prefill": {"ms": round(pre_ms, 3), "tok_s": round(tokens / pre_ms * 1e3, 1), "families": pre_table},
+             "decode": {"ms_per_step": round(dec_ms, 4), "tok_s": round(batch / dec_ms * 1e3, 1),
+                        "graphs": bool(engine.model.graph_safe and a.graph == "on"), "weight_bytes_per_step": nbytes,
+                        "frac_hbm_weights_only": round(nbytes / dec_ms / 1e6 / peaks()["hbm_gbs"], 4), "families": dec_table}}
+    del engine, fn, reqs
+    torch.cuda.empty_cache()
+    return entry
+
+
+def gifopel_compare(a) -> int:
+    """Gifopel beside its closest existing models at equal width, depth, vocabulary, heads and state sizes: a Sebilorn model
+    (attention beside the delta rule where Gifopel has the same, decayed linear attention where Gifopel carries a state, dense
+    feed-forwards) and an LFM2 MoE model (attention and short convolutions, experts of the same size where Gifopel routes).
+    Gifopel's layers repeat: parallel + dense, channel delta + experts, matrix memory + experts, matrix memory + dense. Work:
+    attention 2 (dim + vdim) flops a visible (row, key, head) and, decoding, the bytes of the visible cached rows; a recurrence
+    32-bit flops a (row, head, key, value) on the CUDA cores (8 with the delta rule's read of the state, else 6) and, decoding,
+    the states read and written; the norms the 32-bit rows in and out."""
+    from tandemllm_b200.config import GifopelConfig, Lfm2MoeConfig, SebilornConfig
+    pk = peaks()
+    tokens, batch = a.prefill_tokens, a.batch
+    elem = 2 if a.dtype == "bfloat16" else 4
+    out = []
+    for label in (a.design_sizes.split(",") if a.design_sizes else GIFOPEL_SIZES):
+        z = GIFOPEL_SIZES[label]
+        W, L, V, H, G, D, VD, context, chunk = (z[k] for k in ("width", "layers", "vocab", "heads", "kv", "dim", "vdim", "context", "chunk"))
+        SH, SD, SV = z["s_heads"], z["s_dim"], z["s_vdim"]
+        dense = {"kind": "dense", "ff": z["ff"]}
+        moe = {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"]}, "expert": {"ff": z["expert_ff"]}}
+        rule = {"heads": SH, "kv_heads": z["s_kv"], "dim": SD, "vdim": SV, "conv": 4}
+        memory = {"heads": SH, "dim": SD, "vdim": SV, "gate_cap": 15.0}
+        left = {"heads": H, "kv_heads": G, "dim": D, "vdim": VD, "scale": D ** -0.5, "rot": {"base": 500000.0, "dims": D},
+                "mask": {"size": chunk}}
+        cycle = [("parallel", {"left": left, "right": rule}, dense), ("channel_delta", rule, moe), ("mlstm", memory, moe),
+                 ("mlstm", memory, dense)]
+        gif = GifopelConfig.from_dict({"architecture": "Gifopel", "vocab": V, "width": W, "norm": {"eps": 1e-6}, "layers": [
+            {"type": cycle[i % 4][0], "mixer": cycle[i % 4][1], "mlp": cycle[i % 4][2]} for i in range(L)]})
+        plain_left = {"heads": H, "kv_heads": G, "dim": D, "vdim": VD, "scale": D ** -0.5, "rot": {"base": 1e6, "dims": D}}
+        light = {"heads": SH, "dim": SD, "vdim": SV, "decay": [1.0 - 2.0 ** (-3 - 5 * h / max(SH - 1, 1)) for h in range(SH)]}
+        seb = SebilornConfig.from_dict({"architecture": "Sebilorn", "vocab": V, "width": W, "norm": {"eps": 1e-5},
+                                        "embedding": {"scale": 1.0}, "logit_softcap": 30.0, "layers": [
+            {"type": "parallel", "mlp": dense, "mixer": {"left": plain_left, "right": {"heads": SH, "dim": SD}, "left_scale": 0.5,
+                                                         "right_scale": 0.5}} if i % 4 == 0 else
+            {"type": "lightning", "mlp": dense, "mixer": light} for i in range(L)]})
+        routed = sum(1 for i in range(L) if i % 4 in (1, 2))
+        lfm = Lfm2MoeConfig.from_dict(dict(
+            CONFIG_8B, vocab_size=V, hidden_size=W, intermediate_size=z["ff"], moe_intermediate_size=z["expert_ff"],
+            num_experts=z["experts"], num_experts_per_tok=z["top"], num_hidden_layers=L, num_attention_heads=H,
+            num_key_value_heads=G, head_dim=D, num_dense_layers=L - routed,
+            layer_types=["full_attention" if i % 4 == 0 else "conv" for i in range(L)]))
+        n_par, n_delta, n_mem = (sum(1 for i in range(L) if i % 4 in ks) for ks in ((0,), (1,), (2, 3)))
+        row = {"sizes": dict(z, label=label), "prefill_tokens": tokens, "batch": batch, "context": context}
+        state = float(SH * SD * SV)
+        for name, cfg in (("gifopel", gif), ("sebilorn", seb), ("lfm2_moe_conv_attention", lfm)):
+            entry = time_design(a, cfg, context)
+            chunked = name == "gifopel"
+            pairs = sum(min(i % chunk, i) + 1 for i in range(tokens)) if chunked else tokens * (tokens + 1) // 2
+            seen = (context % chunk or chunk) if chunked else context
+            work = {"attention": (2.0 * (D + VD) * H * pairs * n_par, float(elem) * batch * G * (D + VD) * seen * n_par)}
+            if name == "gifopel":
+                work["gated delta rule (+ convolutions)"] = (8.0 * tokens * state * (n_par + n_delta), 8.0 * batch * state * (n_par + n_delta))
+                work["gated matrix memory"] = (6.0 * tokens * state * n_mem, 8.0 * batch * state * n_mem)
+            elif name == "sebilorn":
+                sq = float(SH * SD * SD)
+                work["matrix-state recurrence"] = (tokens * (10.0 * sq * n_par + 6.0 * state * (L - n_par)),
+                                                   8.0 * batch * (sq * n_par + state * (L - n_par)))
+            # a layer of two norms of one residual: the row in and out, two branches in, two normed rows out; else three rows and one
+            norm_bytes = W * ((4.0 * 4 + 2 * elem) * L if chunked else (4.0 * 3 + elem) * (2 * L + 1))
+            for table, rows_ in ((entry["prefill"]["families"], tokens), (entry["decode"]["families"], batch)):
+                for fam in ("residual add + norm (+ router, + deferred sums)", "residual add + layer norm"):
+                    if fam in table:
+                        rate = norm_bytes * rows_ / table[fam]["ms"] / 1e6
+                        table[fam].update(GBps_rows_only=round(rate, 1), frac_hbm_rows_only=round(rate / pk["hbm_gbs"], 4))
+            for fam, (flops, nbytes) in work.items():
+                pre, dec = entry["prefill"]["families"].get(fam), entry["decode"]["families"].get(fam)
+                if pre:
+                    pre["TFLOPs"] = round(flops / pre["ms"] / 1e9, 2)
+                    if fam == "attention" and a.dtype == "bfloat16":
+                        pre["frac_of_measured_bf16"] = round(flops / pre["ms"] / 1e9 / pk["bf16_tflops"], 4)
+                if dec:
+                    dec["GBps"] = round(nbytes / dec["ms"] / 1e6, 1)
+                    dec["frac_hbm"] = round(nbytes / dec["ms"] / 1e6 / pk["hbm_gbs"], 4)
+            row[name] = entry
+        out.append(row)
+    print(json.dumps({"design_compare": "gifopel beside sebilorn (attention and matrix states, dense) and lfm2 moe (short convolution and attention)",
+                      "dtype": a.dtype, "peaks": pk,
+                      "data": "synthetic: random weights, uniform random token ids, random cached rows as context", "rows": out}))
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1130,16 +1302,18 @@ def main() -> int:
                     help="programmatic dependent launch between the kernels (for comparison; ordinary launches by default)")
     ap.add_argument("--profile", action="store_true",
                     help="bracket the timed decode steps with cudaProfilerStart/Stop (for ncu --profile-from-start off)")
-    ap.add_argument("--design", choices=("sifupel", "puripel", "sebilorn", "niralix"),
+    ap.add_argument("--design", choices=("sifupel", "puripel", "sebilorn", "niralix", "gifopel"),
                     help="measure this design beside the closest existing model at equal layer sizes (its own line)")
     ap.add_argument("--design-sizes", default="", help="--design: which of " + ", ".join(DESIGN_SIZES) + " (sifupel) or "
-                    + ", ".join(PURIPEL_SIZES) + " (puripel) or " + ", ".join(SEBILORN_SIZES) + " (sebilorn) or " + ", ".join(NIRALIX_SIZES) + " (niralix) (default: all)")
+                    + ", ".join(PURIPEL_SIZES) + " (puripel) or " + ", ".join(SEBILORN_SIZES) + " (sebilorn) or " + ", ".join(NIRALIX_SIZES)
+                    + " (niralix) or " + ", ".join(GIFOPEL_SIZES) + " (gifopel) (default: all)")
     a = ap.parse_args()
     if a.impl == "reference":
         return reference_arm(a)
     if a.design:
         a.warmup = max(a.warmup, 3)
-        return {"puripel": puripel_compare, "sebilorn": sebilorn_compare, "niralix": niralix_compare}.get(a.design, design_compare)(a)
+        return {"puripel": puripel_compare, "sebilorn": sebilorn_compare, "niralix": niralix_compare,
+                "gifopel": gifopel_compare}.get(a.design, design_compare)(a)
     if a.gpus != 1:
         print(json.dumps({"error": f"this engine runs on one GPU; --gpus {a.gpus} is not implemented", "n_gpus": a.gpus}))
         return 2

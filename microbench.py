@@ -276,6 +276,49 @@ def recurrence(a) -> dict:
             "ns_per_token_of_a_request": ms * 1e6 / R}
 
 
+def write_recurrence(a) -> dict:
+    """The recurrences whose writes depend on the state or a running maximum, of one layer (`--rule channel`, `head`: the gated delta rule
+    with its convolutions of four taps, two heads a key head; `memory`: the gated matrix memory): `batch` requests of `rows` rows."""
+    import types
+
+    from tandemllm_b200.kernels import ops
+    ops.core()
+    H, D, VD, B, R = a.heads, a.dim, a.vdim, a.batch, a.rows
+    step = types.SimpleNamespace(
+        n_requests=B, max_rows_per_request=R, state_slot=torch.arange(B, dtype=torch.int32, device=DEV),
+        row_start=torch.arange(0, (B + 1) * R, R, dtype=torch.int32, device=DEV),
+        req_of_row=torch.arange(B, dtype=torch.int32, device=DEV).repeat_interleave(R))
+    if a.rule == "memory":
+        cols = {"q": 0, "k": H * D, "v": 2 * H * D, "i": 2 * H * D + H * VD, "f": 2 * H * D + H * VD + H}
+        proj = torch.randn(B * R, cols["f"] + H, device=DEV)
+        slots = torch.zeros(B, H + H * (VD + 1) * D, device=DEV)
+        y, maxima = torch.empty(B * R, H * (VD + 1), device=DEV), torch.empty(B * R, H, device=DEV)
+        bias = torch.zeros(H, device=DEV)
+
+        def run():
+            ops.matrix_memory_scan(proj, cols, bias, bias + 3, 15.0, slots, H, step, y, maxima, H, D, VD, q_scale=D ** -0.5)
+        flops = 6.0
+    else:
+        G = max(1, H // 2)
+        cols = {"q": 0, "k": G * D, "v": 2 * G * D, "b": 2 * G * D + H * VD, "a": 2 * G * D + H * VD + H}
+        proj = torch.randn(B * R, cols["a"] + H, device=DEV)
+        conv, taps = 2 * G * D + H * VD, torch.randn(2 * G * D + H * VD, 4, device=DEV) * 0.5
+        slots = torch.zeros(B, 3 * conv + H * VD * D, device=DEV)
+        y = torch.empty(B * R, H * VD, device=DEV)
+        z = torch.randn(B * R, H * D, device=DEV) if a.rule == "channel" else None
+        dt = torch.full((H * D if a.rule == "channel" else H,), -2.0, device=DEV)
+
+        def run():
+            ops.gated_delta_scan(proj, cols, taps, conv, slots, 3 * conv, step, y, H, G, D, VD, torch.zeros(H, device=DEV), dt,
+                                 unit_eps=1e-6, q_scale=D ** -0.5, decay_logits=z)
+        flops = 8.0
+    ms = timed(run, a.iters)
+    flops *= B * R * H * D * VD
+    nbytes = 4.0 * (proj.numel() + y.numel() + 2 * slots.numel())
+    return {"kernel": f"recurrence ({a.rule})", "batch": B, "rows": R, "heads": H, "dim": D, "vdim": VD, "ms": ms, "flops": flops,
+            "TFLOPs_fp32": flops / ms / 1e9, "bytes": nbytes, "GBps": nbytes / ms / 1e6, "ns_per_token_of_a_request": ms * 1e6 / R}
+
+
 def flex(a) -> dict:
     """Attention with capped scores, a window that keeps first tokens, a turned output and optionally a gate, on the tensor
     cores: `batch` requests of `rows` rows at a context of `context`."""
@@ -360,7 +403,7 @@ def main(argv=None) -> int:
     la.add_argument("--kv-rank", type=int, default=256)
     la.add_argument("--rot-dim", type=int, default=32)
     rc = sub.add_parser("recurrence")
-    rc.add_argument("--rule", default="delta", choices=("delta", "decay", "gated"))
+    rc.add_argument("--rule", default="delta", choices=("delta", "decay", "gated", "channel", "head", "memory"))
     rc.add_argument("--batch", type=int, default=1)
     rc.add_argument("--rows", type=int, default=2048)
     rc.add_argument("--heads", type=int, default=16)
@@ -389,7 +432,8 @@ def main(argv=None) -> int:
         p.add_argument("--iters", type=int, default=20)
     a = ap.parse_args(argv)
     result = {"expert_gemm": expert_gemm, "dense_gemm": dense_gemm, "attention": attention, "norm": norm, "headmix": headmix,
-              "scan": scan, "latent": latent, "recurrence": recurrence, "flex": flex}[a.what](a)
+              "scan": scan, "latent": latent, "flex": flex,
+              "recurrence": write_recurrence if getattr(a, "rule", "") in ("channel", "head", "memory") else recurrence}[a.what](a)
     print(json.dumps({k: (round(v, 4) if isinstance(v, float) else v) for k, v in result.items()}))
     return 0
 

@@ -28,6 +28,16 @@
 
 namespace tl {
 
+constexpr int REC_TOKENS = 8;       // tokens staged at a time: one a warp
+
+// sigmoid(z)^rate without forming the sigmoid: exp(-rate * log(1 + e^-z)), the logarithm split so that neither e^-z nor e^z overflows
+__device__ __forceinline__ float sigmoid_powf_(float z, float rate) {
+  return expf(-rate * (fmaxf(-z, 0.f) + log1pf(expf(-fabsf(z)))));
+}
+
+constexpr int RULE_FIXED = 0, RULE_DELTA = 1, RULE_GATED = 2;
+__host__ __device__ constexpr int rec_arrays(int rule) { return rule == RULE_DELTA ? 5 : (rule == RULE_GATED ? 3 : 2); }
+
 // Dp = 16 P: D rounded up to what P lanes of 16 keys hold. Shared memory: REC_TOKENS x 5 (or 3) arrays of Dp floats, then
 // REC_TOKENS x VD_tile values.
 template <int RULE>
@@ -253,6 +263,193 @@ __global__ void __launch_bounds__(128) recurrence_prepare_kernel(
   }
 }
 
+constexpr int REC_GROUP = 8;
+constexpr int REC_CHUNK = 16;     // the most tokens a stage holds; a column's values of a stage lie this far apart
+// REC_GROUP tokens (FULL) or the first n of them for one lane: the lane's KPL keys of its column go through the tokens, the
+// outputs wait in registers and cross the lanes together. Everything a token needs lies at offsets the compiler knows
+// (`tok`: the lane's first four floats of the group's first prepared token; `vcol`: the column's values, a token a float),
+// so the group is straight-line code whose loads the compiler moves ahead of the chain.
+template <int RULE, int KPL, int DP, bool FULL>
+__device__ __forceinline__ void rec_group(float (&s)[KPL], const float* __restrict__ tok, const float* __restrict__ vcol,
+                                          float* __restrict__ yg, long long ldy, int n, int part, bool owns, float c_h) {
+  constexpr bool DELTA = RULE == RULE_DELTA, GATED = RULE == RULE_GATED;
+  constexpr int P = DP / KPL, M = KPL / 4, tok_floats = rec_arrays(RULE) * DP, Q = DP / 4;
+  float o[REC_GROUP];
+#pragma unroll
+  for (int tt = 0; tt < REC_GROUP; ++tt) {
+    o[tt] = 0.f;
+    if (FULL || tt < n) {
+      const float4* a = reinterpret_cast<const float4*>(tok + tt * tok_floats);
+      const float vj = vcol[tt];
+      float o0 = 0.f, o1 = 0.f, o2 = 0.f, o3 = 0.f;
+      if (DELTA) {
+        float us0 = 0.f, us1 = 0.f, us2 = 0.f, us3 = 0.f;      // four short chains of additions instead of one long one
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+          const float4 u = a[3 * Q + P * m];
+          us0 = fmaf(u.x, s[4 * m], us0);
+          us1 = fmaf(u.y, s[4 * m + 1], us1);
+          us2 = fmaf(u.z, s[4 * m + 2], us2);
+          us3 = fmaf(u.w, s[4 * m + 3], us3);
+        }
+        float us = (us0 + us1) + (us2 + us3);
+#pragma unroll
+        for (int off = P >> 1; off > 0; off >>= 1) us += __shfl_xor_sync(0xffffffffu, us, off);
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+          const float4 q = a[P * m], k = a[Q + P * m], d = a[2 * Q + P * m], au = a[4 * Q + P * m];
+          s[4 * m] = fmaf(d.x, s[4 * m], fmaf(-au.x, us, k.x * vj));
+          s[4 * m + 1] = fmaf(d.y, s[4 * m + 1], fmaf(-au.y, us, k.y * vj));
+          s[4 * m + 2] = fmaf(d.z, s[4 * m + 2], fmaf(-au.z, us, k.z * vj));
+          s[4 * m + 3] = fmaf(d.w, s[4 * m + 3], fmaf(-au.w, us, k.w * vj));
+          o0 = fmaf(s[4 * m], q.x, o0);
+          o1 = fmaf(s[4 * m + 1], q.y, o1);
+          o2 = fmaf(s[4 * m + 2], q.z, o2);
+          o3 = fmaf(s[4 * m + 3], q.w, o3);
+        }
+      } else if (GATED) {
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+          const float4 q = a[P * m], k = a[Q + P * m], d = a[2 * Q + P * m];
+          s[4 * m] = fmaf(d.x, s[4 * m], k.x * vj);
+          s[4 * m + 1] = fmaf(d.y, s[4 * m + 1], k.y * vj);
+          s[4 * m + 2] = fmaf(d.z, s[4 * m + 2], k.z * vj);
+          s[4 * m + 3] = fmaf(d.w, s[4 * m + 3], k.w * vj);
+          o0 = fmaf(s[4 * m], q.x, o0);
+          o1 = fmaf(s[4 * m + 1], q.y, o1);
+          o2 = fmaf(s[4 * m + 2], q.z, o2);
+          o3 = fmaf(s[4 * m + 3], q.w, o3);
+        }
+      } else {
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+          const float4 q = a[P * m], k = a[Q + P * m];
+          s[4 * m] = fmaf(c_h, s[4 * m], k.x * vj);
+          s[4 * m + 1] = fmaf(c_h, s[4 * m + 1], k.y * vj);
+          s[4 * m + 2] = fmaf(c_h, s[4 * m + 2], k.z * vj);
+          s[4 * m + 3] = fmaf(c_h, s[4 * m + 3], k.w * vj);
+          o0 = fmaf(s[4 * m], q.x, o0);
+          o1 = fmaf(s[4 * m + 1], q.y, o1);
+          o2 = fmaf(s[4 * m + 2], q.z, o2);
+          o3 = fmaf(s[4 * m + 3], q.w, o3);
+        }
+      }
+      o[tt] = (o0 + o1) + (o2 + o3);
+    }
+  }
+  rec_reduce_scatter<REC_GROUP, P>(o, part);
+  if (!owns) return;
+  if (P <= REC_GROUP) {
+    constexpr int each = P <= REC_GROUP ? REC_GROUP / P : 1;
+#pragma unroll
+    for (int i = 0; i < each; ++i) {
+      const int t = part * each + i;
+      if (FULL || t < n) yg[t * ldy] = o[i];
+    }
+  } else {
+    constexpr int share = P > REC_GROUP ? P / REC_GROUP : 1;
+    const int t = part / share;
+    if (part % share == 0 && (FULL || t < n)) yg[t * ldy] = o[0];
+  }
+}
+
+// The scan over prepared tokens. Block: cols_per_block * P computing threads (a multiple of 32) and one more warp, the
+// producer, which does nothing but fetch: it keeps STAGES - 1 chunks of TC tokens in flight (each token's NARR * Dp prepared
+// floats, then the chunk's values, a column's REC_CHUNK apart) and meets the computing warps at one barrier a chunk, when the next
+// chunk has landed and the last one has been read.
+// KPL keys of a column a lane (16 or 4): with 4, four times as many lanes share a column and a token takes a warp a
+// third of the instructions, at the price of two more lane crossings a sum; the launcher takes 4 where the GPU would
+// otherwise stand idle. DP: the keys a head, filled up to a power of two (16 at least); sizes known to the compiler keep
+// the loop free of address arithmetic.
+constexpr int REC_STAGES = 3;
+template <int RULE, int KPL, int DP>
+__global__ void __launch_bounds__(REC_THREADS + 32) recurrence_scan_staged_kernel(
+    const float* __restrict__ prep, const float* __restrict__ vsrc, long long ld_v, int v_col, const float* __restrict__ head_decay,
+    float* __restrict__ state, long long slot_floats, const int* __restrict__ state_slot, const int* __restrict__ row_start,
+    float* __restrict__ y, long long rows, int H, int D, int VD, int cols_per_block, int TC, int write_state) {
+  constexpr int STAGES = REC_STAGES, P = DP / KPL, Dp = DP;
+  extern __shared__ __align__(16) float sm[];
+  constexpr int NARR = rec_arrays(RULE);
+  constexpr int M = KPL / 4, tok_floats = NARR * Dp;
+  const int stage_floats = TC * tok_floats + REC_CHUNK * cols_per_block;
+  const int b = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * cols_per_block;
+  const int tid = threadIdx.x, nth = blockDim.x - 32;
+  const bool producer = tid >= nth;
+  const int part = tid % P, jl = tid / P, j = col0 + jl;
+  const bool owns = !producer && j < VD;
+  const int r0 = row_start[b], r1 = row_start[b + 1];
+  if (r1 <= r0) return;
+  float* S = state + (long long)state_slot[b] * slot_floats + (long long)h * D * VD;
+  const float c_h = RULE != RULE_FIXED ? 0.f : head_decay[h];
+  const int n_chunks = (r1 - r0 + TC - 1) / TC;
+
+  // (the producer's lanes only)
+  auto load = [&](int chunk) {
+    const int lane = tid - nth;
+    const int t0 = r0 + chunk * TC, nt = min(TC, r1 - t0);
+    float* base = sm + (chunk % STAGES) * stage_floats;
+    const float* src = prep + ((long long)h * rows + t0) * tok_floats;
+    const int pieces = nt * (tok_floats / 4);
+#pragma unroll 4
+    for (int i = lane; i < pieces; i += 32) rec_cp16(base + 4 * i, src + 4 * i);
+    float* vb = base + TC * tok_floats;
+    const float* vs = vsrc + (long long)t0 * ld_v + v_col + (long long)h * VD + col0;
+    for (int e = lane; e < nt * cols_per_block; e += 32) {
+      const int t = e / cols_per_block, c = e - t * cols_per_block;
+      if (col0 + c < VD) rec_cp4(vb + c * REC_CHUNK + t, vs + (long long)t * ld_v + c);
+      else vb[c * REC_CHUNK + t] = 0.f;
+    }
+  };
+  float s[KPL];
+  if (producer) {
+#pragma unroll
+    for (int s0 = 0; s0 < STAGES - 1; ++s0) {
+      if (s0 < n_chunks) load(s0);
+      asm volatile("cp.async.commit_group;" ::: "memory");
+    }
+    asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");       // chunk 0 has landed
+  } else {
+#pragma unroll
+    for (int m = 0; m < M; ++m)
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        const int i = 4 * (part + P * m) + c;
+        s[4 * m + c] = (owns && i < D) ? S[(long long)i * VD + j] : 0.f;
+      }
+  }
+  __syncthreads();
+
+  for (int chunk = 0; chunk < n_chunks; ++chunk) {
+    if (producer) {
+      // the stage of chunk - 1 is free (everybody passed the barrier behind it): refill it, then wait for chunk + 1
+      if (chunk + STAGES - 1 < n_chunks) load(chunk + STAGES - 1);
+      asm volatile("cp.async.commit_group;" ::: "memory");
+      asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");
+    } else {
+      const int t0 = r0 + chunk * TC, nt = min(TC, r1 - t0);
+      const float* base = sm + (chunk % STAGES) * stage_floats;
+      const float* tok = base + 4 * part;
+      const float* vcol = base + TC * tok_floats + jl * REC_CHUNK;
+      const long long ldy = (long long)H * VD;
+      float* yg = y + (long long)t0 * ldy + (long long)h * VD + j;
+      int g = 0;
+      for (; g + REC_GROUP <= nt; g += REC_GROUP)
+        rec_group<RULE, KPL, DP, true>(s, tok + g * tok_floats, vcol + g, yg + g * ldy, ldy, REC_GROUP, part, owns, c_h);
+      if (g < nt) rec_group<RULE, KPL, DP, false>(s, tok + g * tok_floats, vcol + g, yg + g * ldy, ldy, nt - g, part, owns, c_h);
+    }
+    __syncthreads();
+  }
+  if (write_state && owns) {
+#pragma unroll
+    for (int m = 0; m < M; ++m)
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        const int i = 4 * (part + P * m) + c;
+        if (i < D) S[(long long)i * VD + j] = s[4 * m + c];
+      }
+  }
+}
+
 // grid (rows, groups): out[r, c] = y[r, c] / sqrt(mean over the group of y^2 + eps) * weight[c] * act(gate[r, c]) * scale, act the
 // sigmoid or (silu_gate) g sigmoid(g); with shared_weight the weight has one group's entries, which every group uses
 template <typename T, typename G>
@@ -300,8 +497,20 @@ extern "C" int tl_recurrence_scan(const float* proj, long long ld, int q_col, in
   TL_REQUIRE(H <= 65535, "recurrence_scan: %d heads exceed the grid limit", H);
   int P = 1;
   while (16 * P < D) P <<= 1;
+  const int P16 = P;
   const int sms = sm_count > 0 ? sm_count : 148;
-  const int narr = rec_arrays(rule), Dp = 16 * P;
+  // the staged form gives a column to four times as many lanes (4 keys a lane) until the GPU has two warps a scheduler
+  int kpl = 16;
+  if (scratch && 4 * P <= 32 && (long long)requests * H * VD * P < 256LL * sms) {
+    kpl = 4;
+    P *= 4;
+  }
+  int threads, cols_per_block;
+  recurrence_block(requests, H, VD, P, scratch ? (3LL * sms) / 4 : 2LL * sms, &threads, &cols_per_block);
+  const int tiles = ceil_div(VD, cols_per_block);
+  TL_REQUIRE(tiles <= 65535, "recurrence_scan: %d tiles of value columns exceed the grid limit", tiles);
+  dim3 grid(requests, H, tiles);
+  const int narr = rec_arrays(rule), Dp = 16 * P16;
   if (scratch) {
     const long long pairs = rows * H;
     float* prep = scratch;
@@ -315,20 +524,48 @@ extern "C" int tl_recurrence_scan(const float* proj, long long ld, int q_col, in
     else TL_RPREP(RULE_GATED);
 #undef TL_RPREP
     TL_LAUNCH_CHECK();
+    // tokens a stage: as many (16 at most) as 96 KB hold in three stages
+    int TC = REC_CHUNK;
+    auto bytes = [&](int tc) { return (size_t)REC_STAGES * (tc * narr * Dp + REC_CHUNK * cols_per_block) * sizeof(float); };
+    while (TC > 1 && bytes(TC) > 96 * 1024) TC >>= 1;
+    const size_t smem = bytes(TC);
     const float* vsrc = fixed ? vact : proj;
     const long long ld_v = fixed ? (long long)H * VD : ld;
     const int vc = fixed ? 0 : v_col;
-    const StagedScan a{prep, vsrc, ld_v, vc, head_decay, state, slot_floats, state_slot, row_start, requests, y, rows, H, D, VD,
-                       write_state, sm_count};
-    if (delta) return launch_staged_scan<RULE_DELTA>(a, stream);
-    if (fixed) return launch_staged_scan<RULE_FIXED>(a, stream);
-    return launch_staged_scan<RULE_GATED>(a, stream);
+#define TL_RSS(DELTA_, KPL_, DP_)                                                                                               \
+  do {                                                                                                                          \
+    if (smem > 48 * 1024)                                                                                                       \
+      cudaFuncSetAttribute(recurrence_scan_staged_kernel<DELTA_, KPL_, DP_>, cudaFuncAttributeMaxDynamicSharedMemorySize,       \
+                           96 * 1024);                                                                                          \
+    recurrence_scan_staged_kernel<DELTA_, KPL_, DP_><<<grid, threads + 32, smem, stream>>>(                                     \
+        prep, vsrc, ld_v, vc, head_decay, state, slot_floats, state_slot, row_start, y, rows, H, D, VD, cols_per_block, TC,           \
+        write_state);                                                                                                           \
+  } while (0)
+#define TL_RSS_D(DELTA_, DP_)                   \
+  do {                                          \
+    if (kpl == 16) TL_RSS(DELTA_, 16, DP_);     \
+    else if (DP_ <= 128) TL_RSS(DELTA_, 4, (DP_ <= 128 ? DP_ : 128)); \
+  } while (0)
+#define TL_RSS_ALL(DELTA_)                      \
+  do {                                          \
+    switch (Dp) {                               \
+      case 16: TL_RSS_D(DELTA_, 16); break;     \
+      case 32: TL_RSS_D(DELTA_, 32); break;     \
+      case 64: TL_RSS_D(DELTA_, 64); break;     \
+      case 128: TL_RSS_D(DELTA_, 128); break;   \
+      case 256: TL_RSS_D(DELTA_, 256); break;   \
+      default: TL_RSS_D(DELTA_, 512); break;    \
+    }                                           \
+  } while (0)
+    if (delta) TL_RSS_ALL(RULE_DELTA);
+    else if (fixed) TL_RSS_ALL(RULE_FIXED);
+    else TL_RSS_ALL(RULE_GATED);
+#undef TL_RSS_ALL
+#undef TL_RSS_D
+#undef TL_RSS
+    TL_LAUNCH_CHECK();
+    return 0;
   }
-  int threads, cols_per_block;
-  recurrence_block(requests, H, VD, P, 2LL * sms, &threads, &cols_per_block);
-  const int tiles = ceil_div(VD, cols_per_block);
-  TL_REQUIRE(tiles <= 65535, "recurrence_scan: %d tiles of value columns exceed the grid limit", tiles);
-  dim3 grid(requests, H, tiles);
   const size_t smem = (size_t)(narr * REC_TOKENS * Dp + REC_TOKENS * cols_per_block) * sizeof(float);
 #define TL_RSCAN(RULE_)                                                                                                        \
   do {                                                                                                                         \

@@ -152,7 +152,7 @@ _SIGNATURES = {
     "tl_matrix_memory_scan": [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_float, c_void_p,
                               c_longlong, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                               c_int, c_void_p, c_longlong, c_int, c_void_p],
-    "tl_write_scan_scratch_floats": [c_longlong, c_int, c_int, c_int, c_int],
+    "tl_write_scan_scratch_floats": [c_longlong, c_int, c_int, c_int, c_int, c_int],
     "tl_memory_norm_gate": [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_float, c_float, c_void_p, c_longlong, c_int, c_int,
                             c_int, c_int, c_void_p],
     "tl_group_norm_gate": [c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_float, c_float, c_void_p, c_longlong, c_int,
@@ -910,12 +910,12 @@ def gated_delta_scan(proj, cols: dict, taps, conv_cols: int, slots, state_offset
     `state_offset` floats behind. `y` float32 [rows, heads * value_dim]."""
     _need(proj, torch.float32, "projections"); _need(slots, torch.float32, "slots"); _need(y, torch.float32, "y"); _need(taps, torch.float32, "taps")
     rows = proj.shape[0]
-    rule = 4 if decay_logits is None else 3
+    rule = 1 if decay_logits is None else 0
     if decay_logits is not None and (decay_logits.dtype != torch.float32 or decay_logits.stride(1) != 1):
         raise KernelError("gated delta rule: float32 decay logits with unit stride")
     scratch = None
     if step.max_rows_per_request > RECURRENCE_STAGED_ROWS:
-        scratch = torch.empty(core().tl_write_scan_scratch_floats(rows, heads, key_dim, value_dim, rule), dtype=torch.float32,
+        scratch = torch.empty(core().tl_write_scan_scratch_floats(rows, step.n_requests, heads, key_dim, value_dim, rule), dtype=torch.float32,
                               device=proj.device)
     check(core().tl_gated_delta_scan(
         ptr(proj), proj.stride(0), cols["q"], cols["k"], cols["v"], cols["b"], cols["a"] if decay_logits is None else -1,
@@ -936,7 +936,7 @@ def matrix_memory_scan(proj, cols: dict, i_bias, f_bias, cap: float, slots, stat
     factors = torch.empty(rows, heads, 2, dtype=torch.float32, device=proj.device)
     scratch = None
     if step.max_rows_per_request > RECURRENCE_STAGED_ROWS:
-        scratch = torch.empty(core().tl_write_scan_scratch_floats(rows, heads, key_dim, value_dim + 1, 5), dtype=torch.float32,
+        scratch = torch.empty(core().tl_write_scan_scratch_floats(rows, step.n_requests, heads, key_dim, value_dim + 1, 2), dtype=torch.float32,
                               device=proj.device)
     check(core().tl_matrix_memory_scan(
         ptr(proj), proj.stride(0), cols["q"], cols["k"], cols["v"], cols["i"], cols["f"], ptr(i_bias), ptr(f_bias), float(cap),
