@@ -105,6 +105,91 @@ __global__ void __launch_bounds__(128) qkv_rotate_store_kernel(
   }
 }
 
+template <typename T> struct PairOf;
+template <> struct PairOf<float> { using type = float2; };
+template <> struct PairOf<bf16> { using type = __nv_bfloat162; };
+__device__ __forceinline__ float2 unpack(float2 v) { return v; }
+__device__ __forceinline__ float2 unpack(__nv_bfloat162 v) { return __bfloat1622float2(v); }
+__device__ __forceinline__ void pack_to(float2* p, float a, float b) { *p = make_float2(a, b); }
+__device__ __forceinline__ void pack_to(__nv_bfloat162* p, float a, float b) { *p = __floats2bfloat162_rn(a, b); }
+
+// q/k norms with weights and interleaved pairs (heads of an even size): a warp a head, whose pairs stay in the lanes' registers from
+// the norm to the turn. The same numbers as the kernel above.
+template <typename T>
+__global__ void __launch_bounds__(256) qkv_norm_pairs_store_kernel(
+    const T* __restrict__ qkv, long long ld, int q_col, int k_col, int v_col, const float* __restrict__ inv_freq, int rot,
+    const int* __restrict__ positions, const int* __restrict__ req_of_row, const int* __restrict__ block_table, int max_pages,
+    int page_size, int num_pages, T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache, int Hq, int Hk, int D, int VD,
+    int* __restrict__ status, float rot_magnitude, const float* __restrict__ q_weight, const float* __restrict__ k_weight,
+    float norm_eps) {
+  using T2 = typename PairOf<T>::type;
+  __shared__ float sn[FLEX_MAX_DIM / 2], cs[FLEX_MAX_DIM / 2];
+  const int r = blockIdx.x, lane = threadIdx.x & 31;
+  const int pos = positions[r];
+  const int turned = inv_freq ? rot / 2 : 0, pairs = D / 2;
+  for (int i = threadIdx.x; i < turned; i += blockDim.x) {
+    float s, c;
+    sincosf((float)pos * inv_freq[i], &s, &c);
+    sn[i] = s * rot_magnitude;
+    cs[i] = c * rot_magnitude;
+  }
+  long long at = -1;
+  if (k_col >= 0) {
+    const int page = table_page(block_table + (long long)req_of_row[r] * max_pages, pos / page_size, max_pages, num_pages);
+    if (page < 0) {
+      if (threadIdx.x == 0) atomicExch(status, 2);
+    } else {
+      at = (long long)page * Hk * page_size + pos % page_size;
+    }
+  }
+  __syncthreads();
+  const T* row = qkv + (long long)r * ld;
+  constexpr int HELD = FLEX_MAX_DIM / 64;
+  for (int h = threadIdx.x >> 5; h < Hq + (at >= 0 ? 2 * Hk : 0); h += blockDim.x >> 5) {
+    if (h >= Hq + Hk) {           // a value, as projected
+      const int g = h - Hq - Hk;
+      const T* x = row + v_col + g * VD;
+      T* to = v_cache + (at + (long long)g * page_size) * VD;
+      if ((VD & 1) == 0) {
+        for (int i = lane; i < VD / 2; i += 32) reinterpret_cast<T2*>(to)[i] = reinterpret_cast<const T2*>(x)[i];
+      } else {
+        for (int i = lane; i < VD; i += 32) to[i] = x[i];
+      }
+      continue;
+    }
+    const bool is_q = h < Hq;
+    const int g = is_q ? h : h - Hq;
+    const T2* x = reinterpret_cast<const T2*>(row + (is_q ? q_col : k_col) + g * D);
+    const float2* w = reinterpret_cast<const float2*>(is_q ? q_weight : k_weight);
+    float2 v[HELD];
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < HELD; ++e) {
+      const int i = lane + 32 * e;
+      v[e] = i < pairs ? unpack(x[i]) : make_float2(0.f, 0.f);
+      if (32 * (e + 1) >= pairs) break;
+    }
+#pragma unroll
+    for (int e = 0; e < HELD; ++e) {
+      ss = fmaf(v[e].x, v[e].x, fmaf(v[e].y, v[e].y, ss));
+      if (32 * (e + 1) >= pairs) break;
+    }
+    const float inv = 1.f / sqrtf(warp_sum(ss) / (float)D + norm_eps);
+    T2* to = reinterpret_cast<T2*>(is_q ? q_out + ((long long)r * Hq + g) * D : k_cache + (at + (long long)g * page_size) * D);
+#pragma unroll
+    for (int e = 0; e < HELD; ++e) {
+      const int i = lane + 32 * e;
+      if (i < pairs) {
+        const float2 wi = w[i];
+        const float a = v[e].x * inv * wi.x, b = v[e].y * inv * wi.y;
+        if (i < turned) pack_to(to + i, a * cs[i] - b * sn[i], b * cs[i] + a * sn[i]);
+        else pack_to(to + i, a, b);
+      }
+      if (32 * (e + 1) >= pairs) break;
+    }
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(128) attention_flex_kernel(
     const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
@@ -231,6 +316,20 @@ extern "C" int tl_qkv_rotate_store(const void* qkv, long long ld, int q_col, int
                                                         positions, req_of_row, block_table, max_pages, page_size, num_pages, \
                                                         (T_*)q_out, (T_*)k_cache, (T_*)v_cache, Hq, Hk, D, VD, status,    \
                                                         rot_magnitude, (const T_*)v_other, ld_other, v_blend, q_weight, k_weight, norm_eps, neighbours)
+#define TL_QNP(T_)                                                                                                          \
+  qkv_norm_pairs_store_kernel<T_><<<rows, 256, 0, stream>>>((const T_*)qkv, ld, q_col, k_col, v_col, inv_freq, rot, positions,  \
+                                                            req_of_row, block_table, max_pages, page_size, num_pages, (T_*)q_out, \
+                                                            (T_*)k_cache, (T_*)v_cache, Hq, Hk, D, VD, status, rot_magnitude,   \
+                                                            q_weight, k_weight, norm_eps)
+  // (rows and heads must begin at even entries for the loads in pairs)
+  if (q_weight && (neighbours || !inv_freq) && D % 2 == 0 && !inv_freq_v && !v_other && ld % 2 == 0 && q_col % 2 == 0 &&
+      (k_col < 0 || k_col % 2 == 0) && (k_col < 0 || VD % 2 == 1 || v_col % 2 == 0)) {
+    if (dtype == TL_FP32) TL_QNP(float);
+    else TL_QNP(bf16);
+    TL_LAUNCH_CHECK();
+    return 0;
+  }
+#undef TL_QNP
   if (dtype == TL_FP32) TL_QRS(float);
   else TL_QRS(bf16);
 #undef TL_QRS

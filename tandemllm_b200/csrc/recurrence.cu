@@ -470,6 +470,48 @@ __global__ void group_norm_gate_kernel(const float* __restrict__ y, const G* __r
   }
 }
 
+// The same for groups of up to 256 entries, a warp a (row, group): the group stays in the lanes' registers between the two passes, and
+// its gate and weight are on their way while the squares are summed.
+template <typename T, typename G>
+__global__ void __launch_bounds__(128) group_norm_gate_warp_kernel(const float* __restrict__ y, const G* __restrict__ gate,
+                                                                   long long ld_gate, const float* __restrict__ weight, float eps,
+                                                                   float scale, T* __restrict__ out, long long ld_out, int rows,
+                                                                   int groups, int group, int silu_gate, int shared_weight) {
+  const int lane = threadIdx.x & 31;
+  const long long idx = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+  if (idx >= (long long)rows * groups) return;
+  const long long r = idx / groups;
+  const int c0 = (int)(idx - r * groups) * group;
+  const float* yr = y + r * ((long long)groups * group) + c0;
+  constexpr int HELD = 8;
+  float v[HELD], g[HELD], w[HELD];
+  float ss = 0.f;
+#pragma unroll
+  for (int e = 0; e < HELD; ++e) {
+    const int i = lane + 32 * e;
+    const bool ok = i < group;
+    v[e] = ok ? yr[i] : 0.f;
+    g[e] = ok ? to_f32(gate[r * ld_gate + c0 + i]) : 0.f;
+    w[e] = ok ? weight[(shared_weight ? 0 : c0) + i] : 0.f;
+    if (32 * (e + 1) >= group) break;
+  }
+#pragma unroll
+  for (int e = 0; e < HELD; ++e) {
+    ss = fmaf(v[e], v[e], ss);
+    if (32 * (e + 1) >= group) break;
+  }
+  const float inv = 1.f / sqrtf(warp_sum(ss) / (float)group + eps);
+#pragma unroll
+  for (int e = 0; e < HELD; ++e) {
+    const int i = lane + 32 * e;
+    if (i < group) {
+      const float a = silu_gate ? g[e] / (1.f + expf(-g[e])) : 1.f / (1.f + expf(-g[e]));
+      out[r * ld_out + c0 + i] = from_f32<T>(v[e] * inv * w[e] * a * scale);
+    }
+    if (32 * (e + 1) >= group) break;
+  }
+}
+
 }  // namespace tl
 
 using namespace tl;
@@ -594,14 +636,18 @@ extern "C" int tl_group_norm_gate(const float* y, const void* gate, long long ld
   const int threads = group >= 1024 ? 256 : (group >= 256 ? 128 : (group > 32 ? 64 : 32));
   dim3 grid(rows, groups);
 #define TL_GNG(T_, G_)                                                                                                   \
-  group_norm_gate_kernel<T_, G_><<<grid, threads, 0, stream>>>(y, (const G_*)gate, ld_gate, weight, eps, scale, (T_*)out, \
+  if (group <= 256)                                                                                                      \
+    group_norm_gate_warp_kernel<T_, G_><<<(unsigned)(((long long)rows * groups + 3) / 4), 128, 0, stream>>>(              \
+        y, (const G_*)gate, ld_gate, weight, eps, scale, (T_*)out, ld_out, rows, groups, group, silu_gate, shared_weight); \
+  else                                                                                                                   \
+    group_norm_gate_kernel<T_, G_><<<grid, threads, 0, stream>>>(y, (const G_*)gate, ld_gate, weight, eps, scale, (T_*)out, \
                                                                ld_out, width, group, silu_gate, shared_weight)
   if (dtype == TL_FP32) {
-    if (gate_dtype == TL_FP32) TL_GNG(float, float);
-    else TL_GNG(float, bf16);
+    if (gate_dtype == TL_FP32) { TL_GNG(float, float); }
+    else { TL_GNG(float, bf16); }
   } else {
-    if (gate_dtype == TL_FP32) TL_GNG(bf16, float);
-    else TL_GNG(bf16, bf16);
+    if (gate_dtype == TL_FP32) { TL_GNG(bf16, float); }
+    else { TL_GNG(bf16, bf16); }
   }
 #undef TL_GNG
   TL_LAUNCH_CHECK();

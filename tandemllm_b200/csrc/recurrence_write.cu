@@ -10,8 +10,7 @@
 //                         i = cap tanh((i' + b_i) / cap), f = log sigmoid(cap tanh((f' + b_f) / cap)); m starts at 0. The sum n of
 //                         the keys is carried as one more column of S whose value is always 1: its output is n . q
 //
-// Steps of a few rows a request run one kernel whose blocks prepare up to eight tokens in shared memory, a warp a token, and walk
-// them. The convolution's inputs before the step come from the slot (its last taps - 1 inputs, oldest first); they are moved on by a
+// Steps of a few rows a request run one kernel whose blocks prepare up to eight tokens in shared memory and walk them. The convolution's inputs before the step come from the slot (its last taps - 1 inputs, oldest first); they are moved on by a
 // kernel of their own behind the scan, because the heads that share a key read the same inputs. The running maximum m is a chain
 // over a request's rows in a kernel of its own in front (a warp a request and head), which leaves the two factors of every row.
 //
@@ -84,74 +83,81 @@ __device__ __forceinline__ float conv_silu_at(const TokenParams& p, long long r,
   return siluf_(conv_at<0>(p, r, first, past, c, p.K));
 }
 
-// One warp prepares (row r, head h) into tok (token_floats of it); returns what the head's values are multiplied by.
+// The form for a few rows prepares a token in two passes. First every number of it on its own, `e` from 0 on: the entries of q and k
+// (convolved, not yet of unit length), the decays a key channel, the values of the block's columns from col0 on, and last the write
+// strength and the decay of the whole head. All numbers of a block's tokens are spread over its threads, so that their loads are one
+// round trip to memory.
 template <int RULE>
-__device__ __forceinline__ float prepare_token(const TokenParams& p, long long r, int h, int first, const float* __restrict__ past,
-                                               float* __restrict__ tok, int Dp, int lane) {
+__host__ __device__ constexpr int token_numbers(int Dp, int cols) { return (RULE == WRITE_CHANNEL ? 3 : 2) * Dp + cols + 2; }
+template <int RULE>
+__device__ __forceinline__ void token_number(const TokenParams& p, long long r, int h, int first, const float* __restrict__ past, int e,
+                                             float* __restrict__ tok, float* __restrict__ vals, int Dp, int col0, int cols) {
   const int D = p.D;
-  float* tq = tok;
-  float* tk = tok + Dp;
   float* num = tok + token_arrays(RULE) * Dp;
-  if constexpr (RULE == MEMORY) {
-    const float* q = p.proj + r * p.ld + p.q_col + (long long)h * D;
-    const float* k = p.proj + r * p.ld + p.k_col + (long long)h * D;
-    const float keep = p.factors[(r * p.H + h) * 2], add = p.factors[(r * p.H + h) * 2 + 1];
-    for (int i = lane; i < Dp; i += 32) {
-      tq[i] = i < D ? q[i] * p.q_scale : 0.f;
-      tk[i] = i < D ? k[i] * add : 0.f;
-    }
-    if (lane < 4) num[lane] = lane == 0 ? keep : 0.f;
-    return 1.f;
-  } else {
-    const int g = h / (p.H / p.groups);
-    constexpr int HELD = 512 / 32;              // entries a lane holds of a head of up to 512 keys
-    float q[HELD], k[HELD];
-    float qq = 0.f, kk = 0.f;
-#pragma unroll
-    for (int t = 0; t < HELD; ++t) {
-      const int i = lane + 32 * t;
-      q[t] = k[t] = 0.f;
-      if (i < D) {
-        q[t] = conv_silu_at(p, r, first, past, p.q_col + g * D + i);
-        k[t] = conv_silu_at(p, r, first, past, p.k_col + g * D + i);
-        qq = fmaf(q[t], q[t], qq);
-        kk = fmaf(k[t], k[t], kk);
+  if (e < 2 * Dp) {
+    const bool is_k = e >= Dp;
+    const int i = is_k ? e - Dp : e;
+    float x = 0.f;
+    if (i < D) {
+      if (RULE == MEMORY) {
+        x = p.proj[r * p.ld + (is_k ? p.k_col : p.q_col) + (long long)h * D + i];
+        x *= is_k ? p.factors[(r * p.H + h) * 2 + 1] : p.q_scale;
+      } else {
+        x = conv_silu_at(p, r, first, past, (is_k ? p.k_col : p.q_col) + h / (p.H / p.groups) * D + i);
       }
-      if (32 * (t + 1) >= Dp) break;
     }
-    const float qs = p.q_scale / sqrtf(warp_sum(qq) + p.unit_eps), ks = 1.f / sqrtf(warp_sum(kk) + p.unit_eps);
-    const float beta = sigmoidf_(p.proj[r * p.ld + p.b_col + h]);
-    const float rate = -expf(p.a_log[h]);
-    float d_h = 0.f;
-    if constexpr (RULE == WRITE_HEAD) {
-      d_h = expf(rate * softplusf_(p.proj[r * p.ld + p.a_col + h] + p.dt_bias[h]));
-      if (lane < 4) num[lane] = lane == 0 ? d_h : (lane == 1 ? d_h * beta : 0.f);
+    tok[e] = x;
+    return;
+  }
+  e -= 2 * Dp;
+  if (RULE == WRITE_CHANNEL) {
+    if (e < Dp) {
+      tok[2 * Dp + e] =
+          e < D ? expf(-expf(p.a_log[h]) * softplusf_(p.wl[r * p.ld_w + (long long)h * D + e] + p.dt_bias[h * D + e])) : 0.f;
+      return;
     }
-#pragma unroll
-    for (int t = 0; t < HELD; ++t) {
-      const int i = lane + 32 * t;
-      if (i < Dp) {
-        const float ki = k[t] * ks;
-        tq[i] = q[t] * qs;
-        tk[i] = ki;
-        if constexpr (RULE == WRITE_CHANNEL) {
-          const float d = i < D ? expf(rate * softplusf_(p.wl[r * p.ld_w + (long long)h * D + i] + p.dt_bias[h * D + i])) : 0.f;
-          tok[2 * Dp + i] = d;
-          tok[3 * Dp + i] = beta * (d * ki);
-        }
-      }
-      if (32 * (t + 1) >= Dp) break;
+    e -= Dp;
+  }
+  if (e < cols) {
+    const int j = col0 + e;
+    float x = 0.f;
+    if (j < p.VD) {
+      if (RULE == MEMORY) x = j == p.VD - 1 ? 1.f : p.proj[r * p.ld + p.v_col + (long long)h * (p.VD - 1) + j];
+      else x = conv_silu_at(p, r, first, past, p.v_col + h * p.VD + j);
     }
-    return beta;
+    vals[e] = x;
+    return;
+  }
+  e -= cols;
+  if (RULE == MEMORY) {
+    if (e == 0) num[0] = p.factors[(r * p.H + h) * 2];
+  } else if (e == 1) {
+    num[1] = sigmoidf_(p.proj[r * p.ld + p.b_col + h]);
+  } else if (RULE == WRITE_HEAD) {
+    num[0] = expf(-expf(p.a_log[h]) * softplusf_(p.proj[r * p.ld + p.a_col + h] + p.dt_bias[h]));
   }
 }
-
-// The value of column j of (row r, head h).
+// Then a warp a token: unit lengths, and what the update wants of them.
 template <int RULE>
-__device__ __forceinline__ float token_value(const TokenParams& p, long long r, int h, int first, const float* __restrict__ past,
-                                             int j, float times) {
-  if constexpr (RULE == MEMORY) return j == p.VD - 1 ? 1.f : p.proj[r * p.ld + p.v_col + (long long)h * (p.VD - 1) + j];
-  else return times * conv_silu_at(p, r, first, past, p.v_col + h * p.VD + j);
+__device__ __forceinline__ void finish_token(const TokenParams& p, float* __restrict__ tok, float* __restrict__ vals, int Dp, int cols,
+                                             int lane) {
+  float* num = tok + token_arrays(RULE) * Dp;
+  float qq = 0.f, kk = 0.f;
+  for (int i = lane; i < Dp; i += 32) {
+    qq = fmaf(tok[i], tok[i], qq);
+    kk = fmaf(tok[Dp + i], tok[Dp + i], kk);
+  }
+  const float qs = p.q_scale / sqrtf(warp_sum(qq) + p.unit_eps), ks = 1.f / sqrtf(warp_sum(kk) + p.unit_eps);
+  const float beta = num[1];
+  for (int i = lane; i < Dp; i += 32) {
+    const float k = tok[Dp + i] * ks;
+    tok[i] *= qs;
+    tok[Dp + i] = k;
+    if (RULE == WRITE_CHANNEL) tok[3 * Dp + i] = beta * (tok[2 * Dp + i] * k);
+  }
+  for (int c = lane; c < cols; c += 32) vals[c] *= beta;
+  __syncwarp();
+  if (RULE == WRITE_HEAD && lane == 0) num[1] = num[0] * beta;
 }
 
 // ---- chunks of eight tokens ----
@@ -684,13 +690,18 @@ __global__ void __launch_bounds__(REC_THREADS) write_scan_kernel(TokenParams p, 
   for (int t0 = r0; t0 < r1; t0 += chunk_tokens) {
     const int nt = min(chunk_tokens, r1 - t0);
     __syncthreads();                      // the chunk before has been read
-    if (warp < nt) {
-      const float times = prepare_token<RULE>(p, t0 + warp, h, r0, past, sm + warp * tok_floats, Dp, lane);
-      for (int c = lane; c < cols_per_block; c += 32)
-        s_v[warp * cols_per_block + c] = col0 + c < VD ? token_value<RULE>(p, t0 + warp, h, r0, past, col0 + c, times) : 0.f;
+    const int each = token_numbers<RULE>(Dp, cols_per_block);
+    for (int x = tid; x < nt * each; x += blockDim.x) {
+      const int t = x / each;
+      token_number<RULE>(p, t0 + t, h, r0, past, x - t * each, sm + t * tok_floats, s_v + t * cols_per_block, Dp, col0, cols_per_block);
     }
     __syncthreads();
-    for (int t = 0; t < nt; ++t) {
+    if (RULE != MEMORY) {
+      if (warp < nt) finish_token<RULE>(p, sm + warp * tok_floats, s_v + warp * cols_per_block, Dp, cols_per_block, lane);
+      __syncthreads();
+    }
+    // (warps without columns of their own only help to prepare the tokens)
+    for (int t = 0; t < nt && warp * 32 < cols_per_block * P; ++t) {
       const float4* a = reinterpret_cast<const float4*>(sm + t * tok_floats) + part;
       const float* num = sm + t * tok_floats + token_arrays(RULE) * Dp;
       const int Q = 4 * P;
@@ -797,26 +808,44 @@ __global__ void __launch_bounds__(128) memory_factors_kernel(const float* __rest
   if (write_state && lane == 0) *slot = m;
 }
 
-// grid (rows, heads): o = y / (max(|y_ones|, exp(-maximum)) + floor) with the head's output of the column of ones behind its others,
-// then o / rms(o), times the weight, times sigmoid(gate)
-template <typename T>
-__global__ void memory_norm_gate_kernel(const float* __restrict__ y, const float* __restrict__ maxima, const float* __restrict__ gate,
-                                        long long ld_gate, const float* __restrict__ weight, float eps, float floor_,
-                                        T* __restrict__ out, long long ld_out, int H, int VD) {
-  __shared__ float red[33];
-  const int r = blockIdx.x, h = blockIdx.y;
-  const float* yr = y + ((long long)r * H + h) * (VD + 1);
-  const float inv_den = 1.f / (fmaxf(fabsf(yr[VD]), expf(-maxima[(long long)r * H + h])) + floor_);
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < VD; i += blockDim.x) {
-    const float o = yr[i] * inv_den;
-    ss = fmaf(o, o, ss);
+// A warp a (row, head): o = y / (max(|y_ones|, exp(-maximum)) + floor), the head's output of the column of ones behind its others, then
+// o / rms(o), times the weight, times sigmoid(gate). HELD: entries a lane holds between the passes (VD <= 32 HELD).
+template <typename T, int HELD>
+__global__ void __launch_bounds__(128) memory_norm_gate_kernel(const float* __restrict__ y, const float* __restrict__ maxima,
+                                                               const float* __restrict__ gate, long long ld_gate,
+                                                               const float* __restrict__ weight, float eps, float floor_,
+                                                               T* __restrict__ out, long long ld_out, int rows, int H, int VD) {
+  const int lane = threadIdx.x & 31;
+  const long long idx = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+  if (idx >= (long long)rows * H) return;
+  const long long r = idx / H;
+  const int c0 = (int)(idx - r * H) * VD;
+  const float* yr = y + idx * (VD + 1);
+  float v[HELD], g[HELD], w[HELD];
+  const float ones = yr[VD], maximum = maxima[idx];
+#pragma unroll
+  for (int e = 0; e < HELD; ++e) {
+    const int i = lane + 32 * e;
+    const bool ok = i < VD;
+    v[e] = ok ? yr[i] : 0.f;
+    g[e] = ok ? gate[r * ld_gate + c0 + i] : 0.f;
+    w[e] = ok ? weight[c0 + i] : 0.f;
+    if (32 * (e + 1) >= VD) break;
   }
-  ss = block_sum(ss, red);
-  const float inv = inv_den / sqrtf(ss / (float)VD + eps);
-  for (int i = threadIdx.x; i < VD; i += blockDim.x) {
-    const int c = h * VD + i;
-    out[(long long)r * ld_out + c] = from_f32<T>(yr[i] * inv * weight[c] * sigmoidf_(gate[(long long)r * ld_gate + c]));
+  const float inv_den = 1.f / (fmaxf(fabsf(ones), expf(-maximum)) + floor_);
+  float ss = 0.f;
+#pragma unroll
+  for (int e = 0; e < HELD; ++e) {
+    const float o = v[e] * inv_den;
+    ss = fmaf(o, o, ss);
+    if (32 * (e + 1) >= VD) break;
+  }
+  const float inv = inv_den / sqrtf(warp_sum(ss) / (float)VD + eps);
+#pragma unroll
+  for (int e = 0; e < HELD; ++e) {
+    const int i = lane + 32 * e;
+    if (i < VD) out[r * ld_out + c0 + i] = from_f32<T>(v[e] * inv * w[e] * sigmoidf_(g[e]));
+    if (32 * (e + 1) >= VD) break;
   }
 }
 
@@ -886,6 +915,9 @@ static int write_scan(const TokenParams& p, float* state, float* y, int requests
   const size_t smem = (size_t)(STEP_TOKENS * token_floats(RULE, Dp) + STEP_TOKENS * cols_per_block) * sizeof(float);
   if (smem > 48 * 1024)
     cudaFuncSetAttribute(write_scan_kernel<RULE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  // (enough threads for every number of a token to be asked for at once)
+  const int numbers = ceil_div(token_numbers<RULE>(Dp, cols_per_block), 32) * 32;
+  if (threads < numbers) threads = numbers < REC_THREADS ? numbers : REC_THREADS;
   write_scan_kernel<RULE><<<dim3(requests, p.H, tiles), threads, smem, stream>>>(p, state, y, P, cols_per_block, write_state);
   TL_LAUNCH_CHECK();
   return 0;
@@ -948,14 +980,19 @@ extern "C" int tl_memory_norm_gate(const float* y, const float* maxima, const fl
                                    float eps, float floor_, void* out, long long ld_out, int rows, int H, int VD, int dtype,
                                    cudaStream_t stream) {
   if (rows == 0) return 0;
-  TL_REQUIRE(H > 0 && H <= 65535 && VD > 0, "memory norm: %d heads of %d", H, VD);
-  const int threads = VD > 128 ? 128 : (VD > 32 ? 64 : 32);
-  if (dtype == TL_FP32)
-    memory_norm_gate_kernel<float><<<dim3(rows, H), threads, 0, stream>>>(y, maxima, gate, ld_gate, weight, eps, floor_, (float*)out,
-                                                                          ld_out, H, VD);
-  else
-    memory_norm_gate_kernel<bf16><<<dim3(rows, H), threads, 0, stream>>>(y, maxima, gate, ld_gate, weight, eps, floor_, (bf16*)out,
-                                                                         ld_out, H, VD);
+  TL_REQUIRE(H > 0 && VD > 0 && VD <= 2048, "memory norm: %d heads of %d (up to 2048)", H, VD);
+  const unsigned blocks = (unsigned)(((long long)rows * H + 3) / 4);
+#define TL_MNG(T_, HELD_)                                                                                                   \
+  memory_norm_gate_kernel<T_, HELD_><<<blocks, 128, 0, stream>>>(y, maxima, gate, ld_gate, weight, eps, floor_, (T_*)out, ld_out, \
+                                                                 rows, H, VD)
+  if (dtype == TL_FP32) {
+    if (VD <= 256) TL_MNG(float, 8);
+    else TL_MNG(float, 64);
+  } else {
+    if (VD <= 256) TL_MNG(bf16, 8);
+    else TL_MNG(bf16, 64);
+  }
+#undef TL_MNG
   TL_LAUNCH_CHECK();
   return 0;
 }

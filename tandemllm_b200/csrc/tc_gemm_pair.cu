@@ -386,6 +386,12 @@ __global__ void __launch_bounds__(Smem<GATED, PER_SM>::THREADS, PER_SM) gemm_tc_
               const float neg = fmaf(p.a1, __expf(fminf(z, 0.f)) - 1.f - z, half);
               v[j] = z > 0.f ? fmaf(p.a0 * z, z, half) : neg;
             }
+          } else if (p.unary == TL_ACT_RELU2) {        // (the choice outside the 16 evaluations, as for the gate)
+#pragma unroll
+            for (int j = 0; j < 16; ++j) {
+              const float z = fmaxf(v[j], 0.f);
+              v[j] = z * z;
+            }
           } else if (p.unary) {
 #pragma unroll
             for (int j = 0; j < 16; ++j) v[j] = activation(v[j], p.unary, p.a0, p.a1);
