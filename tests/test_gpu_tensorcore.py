@@ -66,7 +66,7 @@ def test_few_tokens_through_registers_alone(M, N, K):
         ref = want + (0 if bias is None else b)
         assert rel(outs[0], ref) < (1e-2 if out_dtype == torch.bfloat16 else 1e-4), (M, N, K, out_dtype)
     out = torch.empty(M, N, dtype=torch.float32, device=DEV)
-    assert impl.linear(x, wd, None, out) is True and impl._workspace is None, "linear() takes this kernel for such shapes"
+    assert impl.linear(x, wd, None, out) is True and not impl._workspaces, "linear() takes this kernel for such shapes"
     assert not lib.tl_gemm_skinny_supported(33, N, K, K, K) and not lib.tl_gemm_skinny_supported(M, N, K + 4, K + 4, K + 4)
 
 
@@ -205,7 +205,7 @@ def test_split_k_is_used_and_repeatable():
         out = torch.empty(M, N, dtype=torch.float32, device=DEV)
         impl.gemm(x.to(DEV), w.to(DEV), b.to(DEV), out)
         outs.append(out.clone())
-    assert impl._workspace is not None
+    assert impl._workspaces
     assert torch.equal(outs[0], outs[1])
     assert rel(outs[0], x.float() @ w.float().T + b) < 1e-3
 
