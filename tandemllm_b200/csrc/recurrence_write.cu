@@ -10,7 +10,8 @@
 //                         i = cap tanh((i' + b_i) / cap), f = log sigmoid(cap tanh((f' + b_f) / cap)); m starts at 0. The sum n of
 //                         the keys is carried as one more column of S whose value is always 1: its output is n . q
 //
-// Steps of a few rows a request run one kernel whose blocks prepare up to eight tokens in shared memory and walk them. The convolution's inputs before the step come from the slot (its last taps - 1 inputs, oldest first); they are moved on by a
+// Steps of a few rows a request run one kernel whose blocks prepare up to eight tokens in shared memory and walk them. The
+// convolution's inputs before the step come from the slot (its last taps - 1 inputs, oldest first); they are moved on by a
 // kernel of their own behind the scan, because the heads that share a key read the same inputs. The running maximum m is a chain
 // over a request's rows in a kernel of its own in front (a warp a request and head), which leaves the two factors of every row.
 //
