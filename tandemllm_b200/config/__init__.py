@@ -1,5 +1,8 @@
 """Configuration: the typed per-architecture readers, the neutral `ModelSpec`, and the registry."""
 
+from .dipivik import ARCHITECTURES as _DIPIVIK_ARCHS
+from .dipivik import MODEL_TYPES as _DIPIVIK_TYPES
+from .dipivik import DipivikConfig
 from .gifopel import ARCHITECTURES as _GIFOPEL_ARCHS
 from .gifopel import MODEL_TYPES as _GIFOPEL_TYPES
 from .gifopel import GifopelConfig
@@ -20,7 +23,7 @@ from .sebilorn import SebilornConfig
 from .sifupel import ARCHITECTURES as _SIFUPEL_ARCHS
 from .sifupel import MODEL_TYPES as _SIFUPEL_TYPES
 from .sifupel import SifupelConfig
-from .spec import LayerSpec, ModelSpec, PartSpec, Site, StreamAdd, plain_schedule
+from .spec import LayerSpec, ModelSpec, PartSpec, Site, StreamAdd, TokenPairs, plain_schedule
 
 register(Architecture(name="lfm2_moe", architectures=_LFM2_ARCHS, model_types=_LFM2_TYPES,
                       read_config=Lfm2MoeConfig.from_dict))
@@ -40,6 +43,10 @@ register(Architecture(name="niralix", architectures=_NIRALIX_ARCHS, model_types=
 register(Architecture(name="gifopel", architectures=_GIFOPEL_ARCHS, model_types=_GIFOPEL_TYPES,
                       read_config=GifopelConfig.from_dict))
 
-__all__ = ["GifopelConfig", "NiralixConfig", "PuripelConfig", "SebilornConfig", "REGISTRY", "Architecture", "architecture_of", "read_model_config", "register", "unregister",
-           "resolve_model_folder", "spec_of", "LayerSpec", "ModelSpec", "PartSpec", "Site", "StreamAdd", "plain_schedule",
+register(Architecture(name="dipivik", architectures=_DIPIVIK_ARCHS, model_types=_DIPIVIK_TYPES,
+                      read_config=DipivikConfig.from_dict))
+
+__all__ = ["DipivikConfig", "GifopelConfig", "NiralixConfig", "PuripelConfig", "SebilornConfig", "REGISTRY", "Architecture",
+           "architecture_of", "read_model_config", "register", "unregister", "resolve_model_folder", "spec_of", "LayerSpec",
+           "ModelSpec", "PartSpec", "Site", "StreamAdd", "TokenPairs", "plain_schedule",
            "Lfm2MoeConfig", "SifupelConfig"]

@@ -43,7 +43,8 @@ class LayerSpec:
     mixer: PartSpec
     feed_forward: PartSpec
     mixer_norm: PartSpec
-    feed_forward_norm: PartSpec | None          # None: the layer has no feed-forward and no norm for one
+    feed_forward_norm: PartSpec | None          # None: the layer has no feed-forward and no norm for one, or (parallel_residual)
+                                                # mixer and feed-forward both read the mixer's norm
     arrangement: str = "prenorm_residual"
     mixer_post_norm: PartSpec | None = None            # arrangements that norm a branch's output as well
     feed_forward_post_norm: PartSpec | None = None
@@ -56,6 +57,17 @@ class StreamAdd:
     tensor: str
     row: int
     rows: int
+
+
+@dataclass(frozen=True)
+class TokenPairs:
+    """A second embedding, of a token with the one in front of it in its sequence: row (before * mul_prev + token * mul_cur) mod
+    `buckets` of the tensor `tensor` [buckets + 1, hidden] is added to the token's own row; a sequence's first token reads the last
+    row. A request keeps its last token in a slot of its own."""
+    tensor: str
+    buckets: int
+    mul_prev: int
+    mul_cur: int
 
 
 @dataclass(frozen=True)
@@ -80,6 +92,7 @@ class ModelSpec:
     final_norm_prefix: str = field(kw_only=True)    # the last norm's part of its tensors' names
     head_name: str | None = None           # None: the head is the embedding (tied)
     embedding_scale: float = 1.0           # every embedded row is multiplied by this (32-bit)
+    token_pairs: TokenPairs | None = None  # a second embedding added to the first
     logit_scale: float = 1.0               # the head's logits are multiplied by this (32-bit)
     streams: int = 0                       # > 0: the residual is this many streams [streams, rows, hidden] that start as the
                                            # embedded row and are summed in front of the last norm; the layers' arrangement

@@ -23,7 +23,7 @@ struct NormParams {
   long long expert_part_stride;
   const int* pos_of_pair;
   const int* ids;
-  const float* wts;
+  const float* wts;          // null: the expert rows are added as they are
   int top_k;
   const float* weight;
   float eps;
@@ -321,7 +321,7 @@ __global__ void __launch_bounds__(512, (ONE_ROW || MODE == NORM_STREAMS) ? 1 : (
       const bool mine = j < k;
       const int e = mine ? p.ids[(long long)r * k + j] : 0x7fffffff;
       const int src = mine ? p.pos_of_pair[(long long)r * k + j] : 0;
-      const float w = mine ? p.wts[(long long)r * k + j] : 0.f;
+      const float w = mine ? (p.wts ? p.wts[(long long)r * k + j] : 1.f) : 0.f;
       int rank = 0;
       for (int i = 0; i < k; ++i) {
         const int ei = __shfl_sync(0xffffffffu, e, i);
@@ -621,7 +621,7 @@ static int launch_add_rmsnorm(NormParams p, int dtype, cudaStream_t stream) {
   const float* router_w = p.router_w;
   TL_REQUIRE(out_rows > 0 && hidden > 0, "add_rmsnorm: rows %d hidden %d", out_rows, hidden);
   TL_REQUIRE(!p.delta || p.parts >= 1, "add_rmsnorm: %d parts", p.parts);
-  TL_REQUIRE(!p.expert_rows || (p.top_k > 0 && p.top_k <= MAX_TOP_K && p.pos_of_pair && p.ids && p.wts),
+  TL_REQUIRE(!p.expert_rows || (p.top_k > 0 && p.top_k <= MAX_TOP_K && p.pos_of_pair && p.ids),
              "add_rmsnorm: expert rows with top-%d", p.top_k);
   if (router_w) {
     TL_REQUIRE(E > 0 && E <= MAX_EXPERTS, "router: %d experts; up to %d are implemented", E, MAX_EXPERTS);

@@ -6,8 +6,8 @@
 //
 //   latent_prepare    per row: c = w * kv[:L] / rms(kv[:L]) and rot(kv[L:]) go to the request's page at the row's position;
 //                     rot(q_rotated) of every head goes to the query rows q' [rows, H, L + Rr] (32-bit) behind the L
-//                     numbers that head_linear fills. rot: pairs (2i, 2i + 1) of the first `rot_dims` entries turn by
-//                     position * inv_freq[i]; angles, sines and cosines in 32-bit.
+//                     numbers that head_linear fills. rot: pairs (2i, 2i + 1) of the first `rot_dims` entries, or with
+//                     `halves` pairs (i, i + rot_dims / 2), turn by position * inv_freq[i]; angles, sines and cosines in 32-bit.
 //   head_linear       out[r, h, n] = sum_k a[r, h, k] w[h, n, k]: a product a head (q' from q, and the heads' outputs from
 //                     the weighted latents), 32-bit accumulation in a fixed order
 //   attention_latent  per (row, head): softmax over the visible keys j (0 <= pos - j < window, or all) of scale * q' . key_j,
@@ -15,10 +15,23 @@
 //                     to absolute positions, so the order of additions does not depend on how the sequence was cut into
 //                     steps, what else is in the batch or which pages hold the keys. With `sinks` (a number a head) the
 //                     softmax denominator also holds exp(sink): a share of the weight that has no key and no value.
-//                     head_linear may multiply its result entry by entry by sigmoid(gate) (an output gate).
+//                     head_linear may multiply its result by sigmoid(gate), an output gate: a logit an entry or a logit a head.
 #include "common.cuh"
 
 namespace tl {
+
+// Entry i (below rot_dims) of the part of a row at `src`, turned by the row's position.
+template <typename T>
+__device__ __forceinline__ float latent_turned(const T* __restrict__ src, int i, int rot_dims, int halves, float pos,
+                                               const float* __restrict__ inv_freq) {
+  const int half = rot_dims >> 1;
+  const int pair = halves ? (i < half ? i : i - half) : i >> 1;
+  const bool second = halves ? i >= half : (i & 1) != 0;
+  float sn, cs;
+  sincosf(pos * inv_freq[pair], &sn, &cs);
+  const float u = to_f32(src[halves ? pair : i & ~1]), w = to_f32(src[halves ? pair + half : i | 1]);
+  return second ? w * cs + u * sn : u * cs - w * sn;
+}
 
 // grid (rows), 128 threads
 template <typename T>
@@ -26,7 +39,7 @@ __global__ void __launch_bounds__(128) latent_prepare_kernel(
     const T* __restrict__ q, long long ld_q, const T* __restrict__ kv, long long ld_kv, const float* __restrict__ c_weight,
     float eps, const float* __restrict__ inv_freq, int rot_dims, const int* __restrict__ positions,
     const int* __restrict__ req_of_row, const int* __restrict__ table, int max_pages, int page_size, int num_pages,
-    T* __restrict__ cache, float* __restrict__ q_out, int H, int D, int L, int Rr, int* __restrict__ status) {
+    T* __restrict__ cache, float* __restrict__ q_out, int H, int D, int L, int Rr, int halves, int* __restrict__ status) {
   __shared__ float scratch[33];
   const int r = blockIdx.x;
   const int pos = positions[r], b = req_of_row[r];
@@ -50,34 +63,15 @@ __global__ void __launch_bounds__(128) latent_prepare_kernel(
     for (int c = threadIdx.x; c < L; c += blockDim.x) dst[c] = from_f32<T>(to_f32(kvr[c]) * inv * c_weight[c]);
   // the shared key part: pairs of the first rot_dims entries turn, the rest pass
   if (dst)
-    for (int i = threadIdx.x; i < Rr; i += blockDim.x) {
-      float v;
-      if (i < rot_dims) {
-        float sn, cs;
-        sincosf((float)pos * inv_freq[i >> 1], &sn, &cs);
-        const float u = to_f32(kvr[L + (i & ~1)]), w = to_f32(kvr[L + (i | 1)]);
-        v = (i & 1) ? w * cs + u * sn : u * cs - w * sn;
-      } else {
-        v = to_f32(kvr[L + i]);
-      }
-      dst[L + i] = from_f32<T>(v);
-    }
+    for (int i = threadIdx.x; i < Rr; i += blockDim.x)
+      dst[L + i] = from_f32<T>(i < rot_dims ? latent_turned(kvr + L, i, rot_dims, halves, (float)pos, inv_freq) : to_f32(kvr[L + i]));
   // the heads' rotated query parts
   const T* qr = q + (long long)r * ld_q;
   float* qo = q_out + (long long)r * H * Dk;
   for (int i = threadIdx.x; i < H * Rr; i += blockDim.x) {
     const int h = i / Rr, e = i - h * Rr;
     const T* src = qr + (long long)h * (D + Rr) + D;
-    float v;
-    if (e < rot_dims) {
-      float sn, cs;
-      sincosf((float)pos * inv_freq[e >> 1], &sn, &cs);
-      const float u = to_f32(src[e & ~1]), w = to_f32(src[e | 1]);
-      v = (e & 1) ? w * cs + u * sn : u * cs - w * sn;
-    } else {
-      v = to_f32(src[e]);
-    }
-    qo[(long long)h * Dk + L + e] = v;
+    qo[(long long)h * Dk + L + e] = e < rot_dims ? latent_turned(src, e, rot_dims, halves, (float)pos, inv_freq) : to_f32(src[e]);
   }
 }
 
@@ -107,7 +101,7 @@ template <typename T, typename TO>
 __global__ void __launch_bounds__(256) head_linear_kernel(const T* __restrict__ a, long long ld_a, long long a_head,
                                                           const T* __restrict__ w, TO* __restrict__ out, long long ld_out,
                                                           long long out_head, int rows, int N, int K,
-                                                          const T* __restrict__ gate, long long ld_gate) {
+                                                          const T* __restrict__ gate, long long ld_gate, int gate_heads) {
   __shared__ float sA[HL_ROWS][HL_K];
   __shared__ float sW[HL_COLS][HL_K + 1];
   const int h = blockIdx.z, r0 = blockIdx.y * HL_ROWS, n0 = blockIdx.x * HL_COLS;
@@ -136,8 +130,9 @@ __global__ void __launch_bounds__(256) head_linear_kernel(const T* __restrict__ 
     for (int i = 0; i < 4; ++i)
       if (r0 + tr + i < rows) {
         float v = acc[i];
-        // (gate [rows, H * N] logits, rows ld_gate apart: the result times their sigmoid)
-        if (gate) v *= 1.f / (1.f + expf(-to_f32(gate[(long long)(r0 + tr + i) * ld_gate + (long long)h * N + n0 + tn])));
+        // (gate [rows, H * N] logits, or [rows, H] with gate_heads, rows ld_gate apart: the result times their sigmoid)
+        if (gate)
+          v *= 1.f / (1.f + expf(-to_f32(gate[(long long)(r0 + tr + i) * ld_gate + (gate_heads ? (long long)h : (long long)h * N + n0 + tn)])));
         out[(long long)(r0 + tr + i) * ld_out + (long long)h * out_head + n0 + tn] = from_f32<TO>(v);
       }
 }
@@ -267,7 +262,8 @@ using namespace tl;
 extern "C" int tl_latent_prepare(const void* q, long long ld_q, const void* kv, long long ld_kv, const float* c_weight, float eps,
                                  const float* inv_freq, int rot_dims, const int* positions, const int* req_of_row,
                                  const int* table, int max_pages, int page_size, int num_pages, void* cache, float* q_out,
-                                 int rows, int H, int D, int L, int Rr, int dtype, int* status, cudaStream_t stream) {
+                                 int rows, int H, int D, int L, int Rr, int dtype, int* status, int halves,
+                                 cudaStream_t stream) {
   if (rows == 0) return 0;
   TL_REQUIRE(rows > 0 && H > 0 && D >= 0 && L > 0 && Rr >= 0, "latent prepare: %d rows, %d heads of %d + %d, latent %d", rows, H, D,
              Rr, L);
@@ -277,11 +273,11 @@ extern "C" int tl_latent_prepare(const void* q, long long ld_q, const void* kv, 
   if (dtype == TL_FP32)
     latent_prepare_kernel<float><<<rows, 128, 0, stream>>>((const float*)q, ld_q, (const float*)kv, ld_kv, c_weight, eps, inv_freq,
                                                            rot_dims, positions, req_of_row, table, max_pages, page_size,
-                                                           num_pages, (float*)cache, q_out, H, D, L, Rr, status);
+                                                           num_pages, (float*)cache, q_out, H, D, L, Rr, halves, status);
   else
     latent_prepare_kernel<bf16><<<rows, 128, 0, stream>>>((const bf16*)q, ld_q, (const bf16*)kv, ld_kv, c_weight, eps, inv_freq,
                                                           rot_dims, positions, req_of_row, table, max_pages, page_size, num_pages,
-                                                          (bf16*)cache, q_out, H, D, L, Rr, status);
+                                                          (bf16*)cache, q_out, H, D, L, Rr, halves, status);
   TL_LAUNCH_CHECK();
   return 0;
 }
@@ -303,14 +299,14 @@ extern "C" int tl_rmsnorm_rows(const void* in, long long ld_in, const float* w, 
 // `out_dtype`.
 extern "C" int tl_head_linear(const void* a, long long ld_a, long long a_head, const void* w, void* out, long long ld_out,
                               long long out_head, int rows, int H, int N, int K, int dtype, int out_dtype, const void* gate,
-                              long long ld_gate, cudaStream_t stream) {
+                              long long ld_gate, int gate_heads, cudaStream_t stream) {
   if (rows == 0) return 0;
   TL_REQUIRE(rows > 0 && H > 0 && H <= 65535 && N > 0 && K > 0, "head product: %d rows, %d heads, %d x %d", rows, H, N, K);
   TL_REQUIRE(ceil_div(rows, HL_ROWS) <= 65535, "head product: %d rows in one launch", rows);
   const dim3 grid(ceil_div(N, HL_COLS), ceil_div(rows, HL_ROWS), H);
 #define TL_HL(T_, TO_)                                                                                                      \
   head_linear_kernel<T_, TO_><<<grid, 256, 0, stream>>>((const T_*)a, ld_a, a_head, (const T_*)w, (TO_*)out, ld_out, out_head, \
-                                                        rows, N, K, (const T_*)gate, ld_gate)
+                                                        rows, N, K, (const T_*)gate, ld_gate, gate_heads)
   if (dtype == TL_FP32) {
     TL_REQUIRE(out_dtype == TL_FP32, "head product: 32-bit operands give a 32-bit result");
     TL_HL(float, float);

@@ -157,15 +157,20 @@ __device__ __forceinline__ float block_max(float v, float* scratch) {
 #define TL_ACT_CLAMPED_SWISH 6   // a gate form of its own: g' = min(g, a0), u' = clamp(u, -a0, a0); g' sigmoid(a1 g') (u' + 1)
 #define TL_ACT_SOFTCAP 7     // a0 tanh(z / a0): a soft cap on scores or logits (an activation only, never a gate)
 #define TL_ACT_TANH 8        // tanh(z) (an activation only, never a gate)
-#define TL_ACT_GATE_LAST 8   // the last code a gated product's launcher takes
 #define TL_ACT_SCALE 9       // a0 z (an activation only, never a gate)
-#define TL_ACT_LAST 9
+#define TL_ACT_GELU_TANH 10  // the tanh form: 0.5 x (1 + tanh(sqrt(2 / pi) (x + 0.044715 x^3)))
+#define TL_ACT_GATE_LAST 10  // the last code a gated product's launcher takes
+#define TL_ACT_LAST 10
+
+// (1 + tanh(y)) / 2 is the sigmoid of 2 y: what the tanh form of gelu takes it of
+__device__ __forceinline__ float gelu_tanh_argument(float x) { return 1.5957691216057308f * fmaf(0.044715f * x * x, x, x); }
 
 __device__ __forceinline__ float gate_activation(float g, int act) {
   switch (act) {
     case TL_ACT_GELU: return 0.5f * g * (1.f + erff(g * 0.70710678118654752f));
     case TL_ACT_RELU2: { const float r = fmaxf(g, 0.f); return r * r; }
     case TL_ACT_IDENTITY: return g;
+    case TL_ACT_GELU_TANH: return g / (1.f + expf(-gelu_tanh_argument(g)));
     default: return g / (1.f + expf(-g));
   }
 }
@@ -180,6 +185,13 @@ __device__ __forceinline__ float activation(float z, int act, float a0, float a1
   return gate_activation(z, act);
 }
 __device__ __forceinline__ float gated(float g, float u, int act) { return gate_activation(g, act) * u; }
+
+// The grouped products of routed experts may multiply a row by its own weight in front of the expert: expert(w x). The products are
+// linear, so the weight meets the gate's and the up product's sums (32-bit) in front of the activation. `weight` is one number a
+// (row, slot) pair, `index` the pair at every position of the sorted list (null: position i is pair i).
+__device__ __forceinline__ float pair_weight(const float* __restrict__ weight, const int* __restrict__ index, long long position) {
+  return weight ? weight[index ? (long long)index[position] : position] : 1.f;
+}
 // The same with the constants of a gate form that has some (`a0`, `a1`; TL_ACT_CLAMPED_SWISH: the limit and the slope).
 __device__ __forceinline__ float gated(float g, float u, int act, float a0, float a1) {
   if (act == TL_ACT_CLAMPED_SWISH) {

@@ -29,6 +29,8 @@ struct GemmParams {
   const int* n_tiles;      // [1]
   const int* a_gather;     // [M] or nullptr: A row of sorted row i is a_gather[i] / a_div
   int a_div;
+  const float* pair_weight;   // [pairs] or nullptr: the row's weight, applied in front of the activation (gated products)
+  const int* weight_index;    // [M] or nullptr: the pair of sorted row i
   float ga0, ga1;          // the constants of a gate form that has some
   int swiglu;              // a gate activation TL_ACT_* (1: SiLU): W holds 2 N rows per group; C = act(A W[0:N]^T) * (A W[N:2N]^T)
                            // (negative: N rows per group, C = act(A W^T) with the code's activation; grouped products only)
@@ -118,13 +120,14 @@ __global__ void __launch_bounds__(256) gemm_tiled_kernel(GemmParams p) {
     const int lr_out = ty * TM + i;
     if (lr_out >= rows) continue;
     const long long r = row0 + lr_out;
+    const float rw = SWIGLU ? pair_weight(p.pair_weight, p.weight_index, r) : 1.f;
 #pragma unroll
     for (int j = 0; j < TN; ++j) {
       const int n = col0 + tx * TN + j;
       if (n >= p.N) continue;
       float v = acc[i][j];
       if constexpr (SWIGLU) {
-        v = gated(v, acc2[i][j], p.swiglu, p.ga0, p.ga1);
+        v = gated(rw * v, rw * acc2[i][j], p.swiglu, p.ga0, p.ga1);
       } else {
         if (p.bias) v += p.bias[n];
         if (p.swiglu < 0) v = gate_activation(v, -p.swiglu);
@@ -281,22 +284,23 @@ extern "C" int tl_gemm_simt(const void* A, long long lda, const void* W, long lo
 }
 
 // Grouped product over the expert-sorted pair list. Sorted row i multiplies A row (a_gather ? a_gather[i] / a_div : i)
-// by the weights of its tile's expert and writes C row i.
+// by the weights of its tile's expert and writes C row i. `row_weight` and `weight_index` (gated form only): see `pair_weight`.
 extern "C" int tl_gemm_simt_grouped(const void* A, long long lda, const int* a_gather, int a_div, const void* W,
                                     long long ldw, long long w_group_stride, void* C, long long ldc, int n_sorted_rows,
                                     int N, int K, const int* tile_group, const int* tile_row0, const int* tile_rows,
                                     const int* n_tiles, int max_tiles, int swiglu, int in_dtype, int out_dtype,
-                                    cudaStream_t stream) {
+                                    const float* row_weight, const int* weight_index, cudaStream_t stream) {
   if (n_sorted_rows == 0 || N == 0) return 0;
   TL_REQUIRE(n_sorted_rows > 0 && N > 0 && K > 0 && max_tiles > 0, "grouped gemm: rows %d N %d K %d tiles %d",
              n_sorted_rows, N, K, max_tiles);
   TL_REQUIRE(max_tiles <= 65535, "grouped gemm: %d row tiles exceed the grid limit", max_tiles);
   TL_REQUIRE(a_div >= 1, "grouped gemm: a_div %d", a_div);
+  TL_REQUIRE(!row_weight || swiglu > 0, "grouped gemm: row weights need the gated form (activation %d)", swiglu);
   GemmParams p = {};
   p.A = A; p.W = W; p.bias = nullptr; p.C = C; p.lda = lda; p.ldw = ldw; p.ldc = ldc;
   p.w_group_stride = w_group_stride; p.M = n_sorted_rows; p.N = N; p.K = K;
   p.tile_group = tile_group; p.tile_row0 = tile_row0; p.tile_rows = tile_rows; p.n_tiles = n_tiles;
-  p.a_gather = a_gather; p.a_div = a_div; p.swiglu = swiglu;
+  p.a_gather = a_gather; p.a_div = a_div; p.swiglu = swiglu; p.pair_weight = row_weight; p.weight_index = weight_index;
   p.ga0 = tl_gate_constants[0]; p.ga1 = tl_gate_constants[1];
   if (in_dtype == TL_FP32 && out_dtype == TL_FP32) launch<float, float>(p, max_tiles, stream);
   else if (in_dtype == TL_BF16 && out_dtype == TL_BF16) launch<bf16, bf16>(p, max_tiles, stream);

@@ -138,12 +138,14 @@ __global__ void __launch_bounds__(SKINNY_WARPS * 32) gemm_skinny_grouped_kernel(
     long long ldw, long long rows_per_group, TOut* __restrict__ out, long long ldc, int N, int K,
     const int* __restrict__ tile_group, const int* __restrict__ tile_row0, const int* __restrict__ tile_rows,
     const int* __restrict__ n_tiles, const int* __restrict__ pair_group, int n_pairs, int n_groups,
-    int* __restrict__ status, int act, float ga0, float ga1, uint32_t zero) {
+    int* __restrict__ status, int act, float ga0, float ga1, const float* __restrict__ row_weight,
+    const int* __restrict__ weight_index, uint32_t zero) {
   constexpr int W_TILES = SWIGLU ? 2 : 1;
   constexpr int UNROLL = SWIGLU ? 4 : 8;
   __shared__ float part[SKINNY_WARPS][W_TILES][16][8 + 1];
   __shared__ uint32_t s_match[SKINNY_WARPS];
   __shared__ int s_pair[8];
+  __shared__ float s_weight[8];
   chain_next();
   chain_wait();
   const int tile = blockIdx.y;
@@ -219,6 +221,10 @@ __global__ void __launch_bounds__(SKINNY_WARPS * 32) gemm_skinny_grouped_kernel(
   float acc[W_TILES][4];
 #pragma unroll
   for (int j = 0; j < W_TILES; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+  // (a row's own weight, which the epilogue multiplies its sums by, is on its way under the product)
+  float my_weight = 1.f;
+  if constexpr (SWIGLU)
+    if (row_weight && warp == 0 && t == 0 && x_ok) my_weight = pair_weight(row_weight, weight_index, pos);
 
   const int chunks = (K + 31) / 32;
   for (int c0 = warp; c0 < chunks; c0 += SKINNY_WARPS * UNROLL) {
@@ -254,6 +260,7 @@ __global__ void __launch_bounds__(SKINNY_WARPS * 32) gemm_skinny_grouped_kernel(
     part[warp][j][g + 8][2 * t] = acc[j][2];
     part[warp][j][g + 8][2 * t + 1] = acc[j][3];
   }
+  if (SWIGLU && warp == 0 && t == 0) s_weight[g] = my_weight;
   __syncthreads();
   for (int i = threadIdx.x; i < 16 * 8; i += SKINNY_WARPS * 32) {
     const int row = i & 15, m = i >> 4;
@@ -265,7 +272,7 @@ __global__ void __launch_bounds__(SKINNY_WARPS * 32) gemm_skinny_grouped_kernel(
 #pragma unroll
       for (int s = 0; s < SKINNY_WARPS; ++s) v[j] += part[s][j][row][m];
     }
-    const float r = SWIGLU ? gated(v[0], v[W_TILES - 1], act, ga0, ga1) : (act < 0 ? gate_activation(v[0], -act) : v[0]);
+    const float r = SWIGLU ? gated(s_weight[m] * v[0], s_weight[m] * v[W_TILES - 1], act, ga0, ga1) : (act < 0 ? gate_activation(v[0], -act) : v[0]);
     out[(long long)s_pair[m] * ldc + n0 + row] = from_f32<TOut>(r);
   }
 }
@@ -446,12 +453,14 @@ extern "C" int tl_gemm_skinny_mma(const void* x, long long ldx, const void* w, l
 
 // The routed experts of a very small step. x [*, K] bfloat16; w [groups * rows_per_group, K] bfloat16 with, per group, N
 // rows (or, with swiglu, which is then the gate's activation TL_ACT_*, N gate rows then N up rows; negated: N rows whose results go through the activation); the plan's tiles hold at most 8 rows; out [pairs, N] in the plan's
-// order, bfloat16 or 32-bit. row_index (or null) and row_div as in the kernel's comment.
+// order, bfloat16 or 32-bit. row_index (or null) and row_div as in the kernel's comment; row_weight and weight_index (or null; gated
+// form): see `pair_weight`.
 extern "C" int tl_gemm_skinny_grouped(const void* x, long long ldx, const int* row_index, int row_div, const void* w,
                                       long long ldw, long long rows_per_group, void* out, long long ldc, int N, int K,
                                       int swiglu, int out_dtype, const int* tile_group, const int* tile_row0,
                                       const int* tile_rows, const int* n_tiles, int max_tiles, const int* pair_group,
-                                      int n_pairs, int n_groups, int* status, cudaStream_t stream) {
+                                      int n_pairs, int n_groups, int* status, const float* row_weight, const int* weight_index,
+                                      cudaStream_t stream) {
   if (pair_group) max_tiles = n_pairs;
   if (max_tiles == 0 || N == 0) return 0;
   TL_REQUIRE(N >= 1 && K >= 8 && K % 8 == 0 && ldx % 8 == 0 && ldw % 8 == 0 && row_div >= 1 && max_tiles <= 65535,
@@ -463,11 +472,13 @@ extern "C" int tl_gemm_skinny_grouped(const void* x, long long ldx, const int* r
              SKINNY_WARPS * 32);
   TL_REQUIRE(swiglu >= -TL_ACT_IDENTITY && swiglu <= TL_ACT_GATE_LAST,
              "skinny grouped product: gate activation %d is not one of 0..%d (or an ungated one, negated)", swiglu, TL_ACT_GATE_LAST);
+  TL_REQUIRE(!row_weight || swiglu > 0, "skinny grouped product: row weights need the gated form (activation %d)", swiglu);
   const dim3 grid(ceil_div(N, 16), max_tiles), block(SKINNY_WARPS * 32);
 #define TL_GROUPED(SW_, T_)                                                                                              \
   return (int)launch_chained(gemm_skinny_grouped_kernel<SW_, T_>, grid, block, 0, stream, (const bf16*)x, ldx, row_index,  \
                              row_div, (const bf16*)w, ldw, rows_per_group, (T_*)out, ldc, N, K, tile_group, tile_row0,    \
-                             tile_rows, n_tiles, pair_group, n_pairs, n_groups, status, swiglu, tl_gate_constants[0], tl_gate_constants[1], 0u)
+                             tile_rows, n_tiles, pair_group, n_pairs, n_groups, status, swiglu, tl_gate_constants[0], tl_gate_constants[1],     \
+                             row_weight, weight_index, 0u)
   if (swiglu > 0) {
     if (out_dtype == TL_FP32) TL_GROUPED(true, float);
     TL_GROUPED(true, bf16);

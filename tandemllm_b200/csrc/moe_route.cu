@@ -303,7 +303,7 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(const float* __restric
     }
     for (int j = 0; j < k; ++j) {
       s_src[j] = pos_of_pair[(long long)r * k + order[j]];
-      s_w[j] = wts[(long long)r * k + order[j]];
+      s_w[j] = wts ? wts[(long long)r * k + order[j]] : 1.f;      // (no weights: the rows are added as they are)
     }
   }
   __syncthreads();

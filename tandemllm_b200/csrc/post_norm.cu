@@ -52,7 +52,7 @@ __global__ void __launch_bounds__(256) add_normed_kernel(PostNormParams p) {
       const bool mine = j < k;
       const int e = mine ? p.ids[(long long)r * k + j] : 0x7fffffff;
       const int src = mine ? p.pos_of_pair[(long long)r * k + j] : 0;
-      const float w = mine ? p.wts[(long long)r * k + j] : 0.f;
+      const float w = mine ? (p.wts ? p.wts[(long long)r * k + j] : 1.f) : 0.f;
       int rank = 0;
       for (int i = 0; i < k; ++i) {
         const int ei = __shfl_sync(0xffffffffu, e, i);
@@ -239,7 +239,7 @@ extern "C" int tl_add_normed(float* residual, const float* delta, int parts, lon
   TL_REQUIRE(rows > 0 && hidden > 0 && hidden <= 16384, "add_normed: %d rows of %d", rows, hidden);
   TL_REQUIRE(residual && weight && (delta || expert_rows), "add_normed: a residual, a weight and a branch output are needed");
   TL_REQUIRE(!delta || parts >= 1, "add_normed: %d parts", parts);
-  TL_REQUIRE(!expert_rows || (pos_of_pair && ids && wts && top_k > 0 && top_k <= MAX_TOP_K && expert_parts >= 1),
+  TL_REQUIRE(!expert_rows || (pos_of_pair && ids && top_k > 0 && top_k <= MAX_TOP_K && expert_parts >= 1),
              "add_normed: expert rows with top-%d in %d parts", top_k, expert_parts);
   TL_REQUIRE(!pre_weight || normed, "add_normed: the following norm needs a place for its rows");
   TL_REQUIRE(!gather || pre_weight, "add_normed: chosen rows are only read for the following norm");

@@ -7,6 +7,9 @@
 //                            d = sigmoid(w + w0)^rate = exp(-rate * softplus(-(w + w0)))
 //   output                   o = S^T q   with the new S
 //
+// With a fixed decay q and k may be turned by their row's position first (pairs i and i + rot / 2 of the first `rot` entries of a
+// head; angles, sines and cosines in 32-bit) and k multiplied by a constant.
+//
 // and the norm behind them: out = y / rms(y) over each of `groups` equal parts of a row, times a weight, times
 // sigmoid(gate), times a constant.
 //
@@ -35,6 +38,25 @@ __device__ __forceinline__ float sigmoid_powf_(float z, float rate) {
   return expf(-rate * (fmaxf(-z, 0.f) + log1pf(expf(-fabsf(z)))));
 }
 
+// What turns q and k of a fixed decay (rot 0: nothing does).
+struct RecTurn {
+  const int* positions;      // [rows]
+  const float* inv_freq;     // [rot / 2]
+  int rot;
+  float k_scale;
+};
+
+// Entry i (below turn.rot) of q and of k of one head, turned: `q`, `k` its first entries.
+__device__ __forceinline__ void rec_turned(const RecTurn& turn, float pos, const float* __restrict__ q, const float* __restrict__ k,
+                                           int i, float* qv, float* kv) {
+  const int half = turn.rot >> 1, pair = i < half ? i : i - half;
+  float sn, cs;
+  sincosf(pos * turn.inv_freq[pair], &sn, &cs);
+  const float qu = q[pair], qw = q[pair + half], ku = k[pair], kw = k[pair + half];
+  *qv = i < half ? qu * cs - qw * sn : qw * cs + qu * sn;
+  *kv = i < half ? ku * cs - kw * sn : kw * cs + ku * sn;
+}
+
 constexpr int RULE_FIXED = 0, RULE_DELTA = 1, RULE_GATED = 2;
 __host__ __device__ constexpr int rec_arrays(int rule) { return rule == RULE_DELTA ? 5 : (rule == RULE_GATED ? 3 : 2); }
 
@@ -46,7 +68,7 @@ __global__ void __launch_bounds__(REC_THREADS) recurrence_scan_kernel(
     const float* __restrict__ wl, long long ld_w, const float* __restrict__ w0, const float* __restrict__ a_bias,
     const float* __restrict__ head_decay, float rate, float key_eps, int silu_inputs, float q_scale, float* __restrict__ state,
     long long slot_floats, const int* __restrict__ state_slot, const int* __restrict__ row_start, float* __restrict__ y,
-    int H, int D, int VD, int P, int cols_per_block, int write_state) {
+    int H, int D, int VD, int P, int cols_per_block, int write_state, RecTurn turn) {
   extern __shared__ __align__(16) float sm[];
   const int Dp = 16 * P;
   constexpr bool DELTA = RULE == RULE_DELTA, GATED = RULE == RULE_GATED;
@@ -91,15 +113,19 @@ __global__ void __launch_bounds__(REC_THREADS) recurrence_scan_kernel(
       for (int i = lane; i < Dp; i += 32) {
         float qv = 0.f, kv = 0.f;
         if (i < D) {
-          qv = row[q_col + i];
-          kv = row[k_col + i];
+          if (RULE == RULE_FIXED && i < turn.rot) {
+            rec_turned(turn, (float)turn.positions[t0 + tw], row + q_col, row + k_col, i, &qv, &kv);
+          } else {
+            qv = row[q_col + i];
+            kv = row[k_col + i];
+          }
           if (silu_inputs) {
             qv = siluf_(qv);
             kv = siluf_(kv);
           }
         }
         tq[i] = qv * q_scale;
-        tk[i] = kv;
+        tk[i] = RULE == RULE_FIXED ? kv * turn.k_scale : kv;
         ss = fmaf(kv, kv, ss);
       }
       if (DELTA) {
@@ -211,7 +237,7 @@ template <int RULE>
 __global__ void __launch_bounds__(128) recurrence_prepare_kernel(
     const float* __restrict__ proj, long long ld, int q_col, int k_col, int v_col, int a_col, const float* __restrict__ wl,
     long long ld_w, const float* __restrict__ w0, const float* __restrict__ a_bias, float rate, float key_eps, int silu_inputs,
-    float q_scale, float* __restrict__ prep, float* __restrict__ vact, int H, int D, int VD, int Dp, long long pairs) {
+    float q_scale, float* __restrict__ prep, float* __restrict__ vact, int H, int D, int VD, int Dp, long long pairs, RecTurn turn) {
   constexpr bool DELTA = RULE == RULE_DELTA, GATED = RULE == RULE_GATED;
   constexpr int NARR = rec_arrays(RULE);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -226,15 +252,19 @@ __global__ void __launch_bounds__(128) recurrence_prepare_kernel(
   for (int i = lane; i < Dp; i += 32) {
     float qv = 0.f, kv = 0.f;
     if (i < D) {
-      qv = row[q_col + i];
-      kv = row[k_col + i];
+      if (RULE == RULE_FIXED && i < turn.rot) {
+        rec_turned(turn, (float)turn.positions[r], row + q_col, row + k_col, i, &qv, &kv);
+      } else {
+        qv = row[q_col + i];
+        kv = row[k_col + i];
+      }
       if (silu_inputs) {
         qv = siluf_(qv);
         kv = siluf_(kv);
       }
     }
     tq[i] = qv * q_scale;
-    tk[i] = kv;
+    tk[i] = RULE == RULE_FIXED ? kv * turn.k_scale : kv;
     ss = fmaf(kv, kv, ss);
   }
   if (GATED) {
@@ -451,7 +481,8 @@ __global__ void __launch_bounds__(REC_THREADS + 32) recurrence_scan_staged_kerne
 }
 
 // grid (rows, groups): out[r, c] = y[r, c] / sqrt(mean over the group of y^2 + eps) * weight[c] * act(gate[r, c]) * scale, act the
-// sigmoid or (silu_gate) g sigmoid(g); with shared_weight the weight has one group's entries, which every group uses
+// sigmoid or (silu_gate) g sigmoid(g); with shared_weight the weight has one group's entries, which every group uses; without a
+// weight (null) there is none
 template <typename T, typename G>
 __global__ void group_norm_gate_kernel(const float* __restrict__ y, const G* __restrict__ gate, long long ld_gate,
                                        const float* __restrict__ weight, float eps, float scale, T* __restrict__ out,
@@ -466,7 +497,7 @@ __global__ void group_norm_gate_kernel(const float* __restrict__ y, const G* __r
   for (int i = threadIdx.x; i < group; i += blockDim.x) {
     const float g = to_f32(gate[(long long)r * ld_gate + c0 + i]);
     const float a = silu_gate ? g / (1.f + expf(-g)) : 1.f / (1.f + expf(-g));
-    out[(long long)r * ld_out + c0 + i] = from_f32<T>(yr[i] * inv * weight[(shared_weight ? 0 : c0) + i] * a * scale);
+    out[(long long)r * ld_out + c0 + i] = from_f32<T>(yr[i] * inv * (weight ? weight[(shared_weight ? 0 : c0) + i] : 1.f) * a * scale);
   }
 }
 
@@ -492,7 +523,7 @@ __global__ void __launch_bounds__(128) group_norm_gate_warp_kernel(const float* 
     const bool ok = i < group;
     v[e] = ok ? yr[i] : 0.f;
     g[e] = ok ? to_f32(gate[r * ld_gate + c0 + i]) : 0.f;
-    w[e] = ok ? weight[(shared_weight ? 0 : c0) + i] : 0.f;
+    w[e] = ok ? (weight ? weight[(shared_weight ? 0 : c0) + i] : 1.f) : 0.f;
     if (32 * (e + 1) >= group) break;
   }
 #pragma unroll
@@ -524,12 +555,14 @@ extern "C" long long tl_recurrence_scratch_floats(long long rows, int H, int D, 
   return rows * H * (rec_arrays(rule) * 16LL * P + (rule == RULE_FIXED ? VD : 0));
 }
 
+// positions [rows], inv_freq [rot / 2], rot, k_scale: with a fixed decay, see the top of the file (rot 0: nothing turns).
 // scratch: null runs the one-kernel form (steps of a few rows a request); else tl_recurrence_scratch_floats(rows, ...) floats.
 extern "C" int tl_recurrence_scan(const float* proj, long long ld, int q_col, int k_col, int v_col, int a_col, const float* wl,
                                   long long ld_w, const float* w0, const float* a_bias, const float* head_decay, float rate,
                                   float key_eps, int silu_inputs, float* state, long long slot_floats, const int* state_slot,
                                   const int* row_start, int requests, float* y, int H, int D, int VD, int write_state,
-                                  float* scratch, long long rows, int sm_count, int rule, float q_scale, cudaStream_t stream) {
+                                  float* scratch, long long rows, int sm_count, int rule, float q_scale, const int* positions,
+                                  const float* inv_freq, int rot, float k_scale, cudaStream_t stream) {
   if (requests == 0) return 0;
   TL_REQUIRE(rule >= RULE_FIXED && rule <= RULE_GATED, "recurrence_scan: rule %d is not one of 0..2", rule);
   const bool delta = rule == RULE_DELTA, fixed = rule == RULE_FIXED;
@@ -537,6 +570,10 @@ extern "C" int tl_recurrence_scan(const float* proj, long long ld, int q_col, in
   TL_REQUIRE(delta ? (wl && w0 && a_bias && a_col >= 0) : (fixed ? head_decay != nullptr : (wl && w0)),
              "recurrence_scan: the delta rule wants w, w0, a and its bias; the gated rule w and w0; the fixed decay a number a head");
   TL_REQUIRE(H <= 65535, "recurrence_scan: %d heads exceed the grid limit", H);
+  TL_REQUIRE(rot >= 0 && rot <= D && rot % 2 == 0 && (rot == 0 || (fixed && !silu_inputs && positions && inv_freq)),
+             "recurrence_scan: %d turned entries of a head of %d: an even number, with a fixed decay, positions and frequencies", rot, D);
+  TL_REQUIRE(fixed || k_scale == 1.f, "recurrence_scan: a factor on k needs the fixed decay (rule %d)", rule);
+  const RecTurn turn = {positions, inv_freq, rot, k_scale};
   int P = 1;
   while (16 * P < D) P <<= 1;
   const int P16 = P;
@@ -560,7 +597,7 @@ extern "C" int tl_recurrence_scan(const float* proj, long long ld, int q_col, in
     const unsigned pblocks = (unsigned)((pairs + 3) / 4);
 #define TL_RPREP(RULE_)                                                                                                          \
   recurrence_prepare_kernel<RULE_><<<pblocks, 128, 0, stream>>>(proj, ld, q_col, k_col, v_col, a_col, wl, ld_w, w0, a_bias, rate, \
-                                                                key_eps, silu_inputs, q_scale, prep, vact, H, D, VD, Dp, pairs)
+                                                                key_eps, silu_inputs, q_scale, prep, vact, H, D, VD, Dp, pairs, turn)
     if (delta) TL_RPREP(RULE_DELTA);
     else if (fixed) TL_RPREP(RULE_FIXED);
     else TL_RPREP(RULE_GATED);
@@ -616,7 +653,7 @@ extern "C" int tl_recurrence_scan(const float* proj, long long ld, int q_col, in
     recurrence_scan_kernel<RULE_><<<grid, threads, smem, stream>>>(proj, ld, q_col, k_col, v_col, a_col, wl, ld_w, w0, a_bias, \
                                                                    head_decay, rate, key_eps, silu_inputs, q_scale, state,     \
                                                                    slot_floats, state_slot, row_start, y, H, D, VD, P,         \
-                                                                   cols_per_block, write_state);                               \
+                                                                   cols_per_block, write_state, turn);                         \
   } while (0)
   if (delta) TL_RSCAN(RULE_DELTA);
   else if (fixed) TL_RSCAN(RULE_FIXED);

@@ -1,4 +1,4 @@
-// Row-wise kernels: embedding gather, residual add fused with RMS norm (and, for the rows of an expert layer, with
+// Row-wise kernels: embedding gather (with a second table over pairs of tokens), residual add fused with RMS norm (and, for the rows of an expert layer, with
 // the router), SwiGLU gating, and the last error message of the library.
 //
 // The residual stream is 32-bit in both precisions; norms compute mean(x^2), rsqrt and the scale in
@@ -42,6 +42,49 @@ __global__ void embed_rows_kernel(const T* __restrict__ table, const int* __rest
   }
 }
 
+// residual[r, :] = float(table[t, :]) * scale + float(pairs[row, :]), t the row's token and row = (before * mul_prev + t * mul_cur)
+// mod buckets, `before` the token in front of it in its sequence; a sequence's first token reads row `buckets`. Inside a portion the
+// token in front is the row before; a portion's first row finds it in the request's slot (last_token; negative: there is none), and
+// leaves the portion's last token there once it has read it. No other block touches the slot.
+template <typename T>
+__global__ void embed_token_pairs_kernel(const T* __restrict__ table, const T* __restrict__ pairs, const int* __restrict__ tokens,
+                                         const int* __restrict__ req_of_row, const int* __restrict__ row_start,
+                                         const int* __restrict__ state_slot, int* __restrict__ last_token,
+                                         float* __restrict__ residual, int hidden, int vocab, long long buckets, long long mul_prev,
+                                         long long mul_cur, int* __restrict__ status, float scale) {
+  __shared__ long long s_row;
+  chain_next();
+  chain_wait();
+  const int r = blockIdx.x;
+  int tok = tokens[r];
+  if (tok < 0 || tok >= vocab) {
+    if (threadIdx.x == 0) atomicExch(status, 1);   // recorded, and the row reads token 0 instead of faulting
+    tok = 0;
+  }
+  if (threadIdx.x == 0) {
+    const int b = req_of_row[r], first = row_start[b];
+    int before;
+    if (r == first) {
+      int* slot = last_token + state_slot[b];
+      before = *slot;
+      *slot = tokens[row_start[b + 1] - 1];
+    } else {
+      before = tokens[r - 1];
+    }
+    long long at = buckets;
+    if (before >= 0) {
+      at = ((long long)before * mul_prev + (long long)tok * mul_cur) % buckets;
+      if (at < 0) at += buckets;
+    }
+    s_row = at;
+  }
+  __syncthreads();
+  const T* src = table + (size_t)tok * hidden;
+  const T* pair = pairs + (size_t)s_row * hidden;
+  float* dst = residual + (size_t)r * hidden;
+  for (int c = threadIdx.x; c < hidden; c += blockDim.x) dst[c] = to_f32(src[c]) * scale + to_f32(pair[c]);
+}
+
 // out[r, i] = act(gate_up[r, i]) * gate_up[r, inter + i]
 template <typename T>
 __global__ void silu_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ out, long long rows, int inter, int act,
@@ -81,6 +124,26 @@ extern "C" int tl_embed_rows_copies(const void* table, const int* tokens, float*
 extern "C" int tl_embed_rows(const void* table, const int* tokens, float* residual, int rows, int hidden, int vocab,
                              int dtype, int* status, float scale, cudaStream_t stream) {
   return tl_embed_rows_copies(table, tokens, residual, rows, hidden, vocab, dtype, status, scale, 1, 0, stream);
+}
+
+// pairs [buckets + 1, hidden] of the table's type; last_token [slots]. See embed_token_pairs_kernel.
+extern "C" int tl_embed_token_pairs(const void* table, const void* pairs, const int* tokens, const int* req_of_row,
+                                    const int* row_start, const int* state_slot, int* last_token, float* residual, int rows,
+                                    int hidden, int vocab, long long buckets, long long mul_prev, long long mul_cur, int dtype,
+                                    int* status, float scale, cudaStream_t stream) {
+  if (rows == 0) return 0;
+  TL_REQUIRE(rows > 0 && hidden > 0 && vocab > 0 && buckets > 0, "embed_token_pairs: rows %d hidden %d vocab %d buckets %lld", rows,
+             hidden, vocab, buckets);
+  TL_REQUIRE(table && pairs && req_of_row && row_start && state_slot && last_token, "embed_token_pairs: two tables, the rows' requests "
+             "and a slot a request are needed (%d rows)", rows);
+  const int threads = hidden >= 1024 ? 256 : 128;
+#define TL_PAIRS(T_)                                                                                                            \
+  return (int)launch_chained(embed_token_pairs_kernel<T_>, dim3(rows), dim3(threads), 0, stream, (const T_*)table,              \
+                             (const T_*)pairs, tokens, req_of_row, row_start, state_slot, last_token, residual, hidden, vocab,  \
+                             buckets, mul_prev, mul_cur, status, scale)
+  if (dtype == TL_FP32) TL_PAIRS(float);
+  TL_PAIRS(bf16);
+#undef TL_PAIRS
 }
 
 extern "C" void tl_set_chained_launches(int enabled) { chained_launches() = enabled; }

@@ -49,6 +49,8 @@ struct TcParams {
   int act;                    // the gate's activation of a gated product (TL_ACT_*), 0 for a plain one; negated: an activation
                               // on a plain product's results
   float ga0, ga1;             // the constants of a gate form that has some
+  const float* row_weight;    // grouped, gated (or nullptr): a (row, slot) pair's own weight, see `pair_weight`
+  const int* weight_index;    // the pair at every position of the sorted list (nullptr: position i is pair i)
   int skip_kb;                // -1; a test sets the k-block whose copies the producer leaves out, so that a wait runs out
   int* status;
 };
@@ -315,7 +317,8 @@ __global__ void __launch_bounds__(192) gemm_tc_kernel(const __grid_constant__ CU
             for (int j = 0; j < 16; ++j) {
               const int t = c0 + j;
               if (t < tok_rows) {
-                const float r = SWIGLU ? gated(v[j], u[j], p.act, p.ga0, p.ga1) : plain_result(v[j] + b, p.act);
+                const float rw = SWIGLU ? pair_weight(p.row_weight, p.weight_index, tok0 + t) : 1.f;
+                const float r = SWIGLU ? gated(rw * v[j], rw * u[j], p.act, p.ga0, p.ga1) : plain_result(v[j] + b, p.act);
                 if (p.partial) p.partial[((long long)blockIdx.z * p.M + tok0 + t) * p.N + n] = r;
                 else store_out<TOut>(C + (long long)(tok0 + t) * p.ldc + n, r);
               }
@@ -325,11 +328,12 @@ __global__ void __launch_bounds__(192) gemm_tc_kernel(const __grid_constant__ CU
           // this thread: token tok0 + m_row; registers: output columns n0 + c0 + j
           if (m_row < tok_rows) {
             TOut* row = C + (long long)(tok0 + m_row) * p.ldc;
+            const float rw = SWIGLU ? pair_weight(p.row_weight, p.weight_index, tok0 + m_row) : 1.f;
             float r[16];
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
               const int n = n0 + c0 + j;
-              r[j] = SWIGLU ? gated(v[j], u[j], p.act, p.ga0, p.ga1)
+              r[j] = SWIGLU ? gated(rw * v[j], rw * u[j], p.act, p.ga0, p.ga1)
                             : plain_result(v[j] + ((p.bias && n < p.N) ? p.bias[n] : 0.f), p.act);
             }
             // 16 consecutive outputs of one row: 16-byte stores when they are all there and aligned
@@ -535,11 +539,12 @@ __global__ void __launch_bounds__(192) gemm_tc_persistent_kernel(const __grid_co
           for (int j = 0; j < 16; ++j) v[j] = u[j] = 0.f;
         }
         if (m_row < tok_rows && n0 + c0 < p.N) {
+          const float rw = SWIGLU ? pair_weight(p.row_weight, p.weight_index, tok0 + m_row) : 1.f;
           float r[16];
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
             const int col = n0 + c0 + j;
-            r[j] = SWIGLU ? gated(v[j], u[j], p.act, p.ga0, p.ga1)
+            r[j] = SWIGLU ? gated(rw * v[j], rw * u[j], p.act, p.ga0, p.ga1)
                           : plain_result(v[j] + ((p.bias && col < p.N) ? p.bias[col] : 0.f), p.act);
           }
           const bool whole = n0 + c0 + 16 <= p.N && (((uintptr_t)(row + n0 + c0)) & 15) == 0;
@@ -677,12 +682,14 @@ extern "C" int tl_tc_token_tile(int swap, int bn) { return swap ? bn : TILE_M; }
 // swiglu: W holds 2 N rows per group (gate then up) and C = act(gate) * up; a negated code: N rows and C = act(X W^T). out_dtype: TL_BF16 or TL_FP32.
 // splits > 1 (swap, not swiglu): `partial` must hold splits * M * N floats; a grouped product leaves the sums to the caller.
 // row_index (swap, grouped; or null): the tile map's rows are positions of this list, and position i stands for row
-// row_index[i] / row_div of X; without it X itself is in the tile map's order.
+// row_index[i] / row_div of X; without it X itself is in the tile map's order. row_weight, weight_index (grouped and gated, or
+// null): see `pair_weight`.
 extern "C" int tl_gemm_tc(const void* X, long long ldx, long long x_rows, const void* W, long long ldw, long long w_rows,
                           long long rows_per_group, const float* bias, void* C, long long ldc, int M, int N, int K, int swap,
                           int bn, int swiglu, int out_dtype, const int* tile_group, const int* tile_row0,
                           const int* tile_rows, const int* n_tiles, int max_tiles, const int* row_index, int row_div,
-                          int splits, float* partial, int reduce, int* status, cudaStream_t stream) {
+                          int splits, float* partial, int reduce, int* status, const float* row_weight, const int* weight_index,
+                          cudaStream_t stream) {
   if (M == 0 || N == 0) return 0;
   TL_REQUIRE(M > 0 && N > 0 && K > 0, "tensor-core gemm: M %d N %d K %d", M, N, K);
   TL_REQUIRE(K % 8 == 0 && ldx % 8 == 0 && ldw % 8 == 0,
@@ -693,6 +700,7 @@ extern "C" int tl_gemm_tc(const void* X, long long ldx, long long x_rows, const 
   TL_REQUIRE(splits >= 1 && (splits == 1 || (swap && !swiglu && partial && (!tile_group || !reduce))),
              "tensor-core gemm: split-K needs the swapped plain kernel and a workspace (grouped: the caller adds the sums)");
   const bool gated_form = swiglu > 0;
+  TL_REQUIRE(!row_weight || (gated_form && tile_group), "tensor-core gemm: row weights need the grouped, gated form (%d)", swiglu);
   TL_REQUIRE(!bias || !swiglu, "tensor-core gemm: a bias with the gated epilogue is not implemented");
   TL_REQUIRE(swiglu >= -TL_ACT_IDENTITY && swiglu <= TL_ACT_GATE_LAST,
              "tensor-core gemm: gate activation %d is not one of 0..%d (or an ungated one, negated)", swiglu, TL_ACT_GATE_LAST);
@@ -710,7 +718,7 @@ extern "C" int tl_gemm_tc(const void* X, long long ldx, long long x_rows, const 
   p.rows_per_group = rows_per_group;
   p.tile_group = tile_group; p.tile_row0 = tile_row0; p.tile_rows = tile_rows; p.n_tiles = n_tiles; p.status = status;
   p.row_index = row_index; p.row_div = row_index ? row_div : 1;
-  p.act = swiglu;
+  p.act = swiglu; p.row_weight = row_weight; p.weight_index = weight_index;
   p.ga0 = tl_gate_constants[0]; p.ga1 = tl_gate_constants[1];
   p.skip_kb = skip_kb_for_test();
   const int tok_tile = swap ? bn : TILE_M, n_tile = swap ? TILE_M : bn;

@@ -51,6 +51,8 @@ struct Params {
   int unary;                  // plain product: an activation (TL_ACT_*) applied to every output (after the bias), 0 for none
   float a0, a1;               // that activation's constants
   float ga0, ga1;             // the constants of a gate form that has some
+  const float* row_weight;    // grouped, gated (or nullptr): a (row, slot) pair's own weight, see `pair_weight`
+  const int* weight_index;    // the pair at every position of the sorted list (nullptr: position i is pair i)
   int skip_kb;                // -1; a test sets the k-block (counted over a cluster's tiles) whose copies both producers leave out
   int splits;                 // plain, ungrouped: work items a tile, each a run of k-blocks with a 32-bit partial result of its own
   int kb_per_split;           // k-blocks a run (every run holds at least one)
@@ -347,12 +349,16 @@ __global__ void __launch_bounds__(Smem<GATED, PER_SM>::THREADS, PER_SM) gemm_tc_
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       const uint32_t taddr = tmem_base + ((uint32_t)(quad * 32) << 16) + buf * 256;
       const int col = n0 + (int)rank * ROWS + m_row;                 // this thread's output
-      const float b = (!GATED && p.bias && col < p.N && kb0 == 0) ? p.bias[col] : 0.f;
+      const float b = (p.bias && col < p.N && kb0 == 0) ? p.bias[col] : 0.f;
+      const float b_up = (GATED && p.bias && col < p.N) ? p.bias[p.N + col] : 0.f;      // (gated: N gate biases, then N of the up rows)
       const int j_tok = lane >> 1, c_half = (lane & 1) * 16;        // after the turn: token c0 + j_tok, 16 outputs
       const int out0 = n0 + (int)rank * ROWS + quad * 32 + c_half;
 #pragma unroll 1
       for (int c0 = 16 * turn_of; c0 < n_mma; c0 += 16 * (S::EPI_WARPS / 4)) {
         float v[16], u[16];
+        float rw = 1.f;                                              // lane j: the weight of token c0 + j's pair
+        if (GATED && p.row_weight && c0 + (lane & 15) < tok_rows)
+          rw = pair_weight(p.row_weight, p.weight_index, (long long)tok0 + c0 + (lane & 15));
         if (num_kb > 0) {
           ld16(taddr + c0, v);
           if (GATED) ld16(taddr + S::UP_COL + c0, u);
@@ -367,9 +373,27 @@ __global__ void __launch_bounds__(Smem<GATED, PER_SM>::THREADS, PER_SM) gemm_tc_
           // The gated product's MMAs wait for this loop, so it is written for speed: the choice of the activation
           // stands outside the 16 independent evaluations, and SiLU, the usual one, takes the fast exponential and
           // division (the result is rounded to bfloat16, far coarser than their error).
+          if (p.row_weight) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) {
+              const float wj = __shfl_sync(0xffffffffu, rw, j);
+              v[j] *= wj;
+              u[j] *= wj;
+            }
+          }
+          if (p.bias) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) {
+              v[j] += b;
+              u[j] += b_up;
+            }
+          }
           if (p.act == TL_ACT_SILU) {
 #pragma unroll
             for (int j = 0; j < 16; ++j) v[j] = __fdividef(v[j], 1.f + __expf(-v[j])) * u[j];
+          } else if (p.act == TL_ACT_GELU_TANH) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) v[j] = __fdividef(v[j], 1.f + __expf(-gelu_tanh_argument(v[j]))) * u[j];
           } else {
 #pragma unroll
             for (int j = 0; j < 16; ++j) v[j] = gated(v[j], u[j], p.act, p.ga0, p.ga1);
@@ -520,7 +544,8 @@ extern "C" int tl_tc_pair_resident(int gated, int per_sm) {
 
 // X [M, K] (row stride ldx, x_rows rows in the tensor), W [groups * rows_per_group, K] (row stride ldw). Plain: groups = 1,
 // tile_group = nullptr. gated (an activation code TL_ACT_*, or 0): W holds 2 N rows per group (gate then up) and
-// C = act(gate) * up; a negated code: N rows and C = act(X W^T). out_dtype: TL_BF16 or TL_FP32. Grouped: the tile map's tiles hold at most tl_tc_pair_token_tile()
+// C = act(gate) * up (`bias`, ungrouped: 2 N numbers in the same order); a negated code: N rows and C = act(X W^T). row_weight,
+// weight_index (grouped and gated, or null): see `pair_weight`. out_dtype: TL_BF16 or TL_FP32. Grouped: the tile map's tiles hold at most tl_tc_pair_token_tile()
 // rows (plan_rows: the height the map was built with). per_sm: 1 or 2 CTAs an SM (see Smem). splits > 1 (plain, ungrouped,
 // 32-bit output): the reduction is cut into `splits` runs of k-blocks, each a work item of its own, and C receives the
 // runs' partial results one behind the other, [splits, M, ldc], for the caller to add in order (a product with fewer
@@ -529,7 +554,7 @@ static int pair_product(const void* X, long long ldx, long long x_rows, const vo
                         long long rows_per_group, const float* bias, void* C, long long ldc, int M, int N, int K,
                         int gated, int out_dtype, const int* tile_group, const int* tile_row0, const int* tile_rows,
                         const int* n_tiles, int max_tiles, int plan_rows, int per_sm, int splits, int unary, float a0, float a1,
-                        int* status, cudaStream_t stream) {
+                        int* status, const float* row_weight, const int* weight_index, cudaStream_t stream) {
   if (M == 0 || N == 0) return 0;
   TL_REQUIRE(unary >= 0 && unary <= TL_ACT_LAST && (!unary || (!gated && splits == 1)),
              "pair product: an activation on the outputs (%d) needs the plain product in one run", unary);
@@ -538,7 +563,8 @@ static int pair_product(const void* X, long long ldx, long long x_rows, const vo
              "pair product: K %d and the row strides %lld, %lld must be multiples of 8 elements (16 bytes) for TMA", K, ldx, ldw);
   TL_REQUIRE(((uintptr_t)X & 15) == 0 && ((uintptr_t)W & 15) == 0, "pair product: operands must be 16-byte aligned (%d)", 0);
   TL_REQUIRE(out_dtype == TL_BF16 || out_dtype == TL_FP32, "pair product: output dtype %d", out_dtype);
-  TL_REQUIRE(!bias || !gated, "pair product: a bias with the gated epilogue is not implemented (%d)", gated);
+  TL_REQUIRE(!bias || !gated || !tile_group, "pair product: a bias with the grouped, gated form is not implemented (%d)", gated);
+  TL_REQUIRE(!row_weight || (gated && tile_group), "pair product: row weights need the grouped, gated form (%d)", gated);
   TL_REQUIRE(gated >= 0 && gated <= TL_ACT_GATE_LAST, "pair product: gate activation %d is not one of 0..%d", gated, TL_ACT_GATE_LAST);
   TL_REQUIRE(!tile_group || (tile_row0 && tile_rows && n_tiles && max_tiles > 0 && plan_rows > 0),
              "pair product: incomplete tile map (tiles of %d rows)", plan_rows);
@@ -561,7 +587,7 @@ static int pair_product(const void* X, long long ldx, long long x_rows, const vo
   p.rows_per_group = rows_per_group;
   p.tile_group = tile_group; p.tile_row0 = tile_row0; p.tile_rows = tile_rows; p.n_tiles = n_tiles;
   p.plan_rows = plan_rows;
-  p.act = gated; p.status = status;
+  p.act = gated; p.status = status; p.row_weight = row_weight; p.weight_index = weight_index;
   p.ga0 = tl_gate_constants[0]; p.ga1 = tl_gate_constants[1];
   p.unary = unary; p.a0 = a0; p.a1 = a1;
   p.skip_kb = pair::skip_kb_for_test();
@@ -578,10 +604,10 @@ extern "C" int tl_gemm_tc_pair(const void* X, long long ldx, long long x_rows, c
                                long long rows_per_group, const float* bias, void* C, long long ldc, int M, int N, int K,
                                int gated, int out_dtype, const int* tile_group, const int* tile_row0, const int* tile_rows,
                                const int* n_tiles, int max_tiles, int plan_rows, int per_sm, int splits, int* status,
-                               cudaStream_t stream) {
+                               const float* row_weight, const int* weight_index, cudaStream_t stream) {
   return pair_product(X, ldx, x_rows, W, ldw, w_rows, rows_per_group, bias, C, ldc, M, N, K, gated > 0 ? gated : 0, out_dtype,
                       tile_group, tile_row0, tile_rows, n_tiles, max_tiles, plan_rows, per_sm, splits, gated < 0 ? -gated : 0, 0.f,
-                      0.f, status, stream);
+                      0.f, status, row_weight, weight_index, stream);
 }
 
 // C = act(X W^T + bias): the plain, ungrouped product with an activation (TL_ACT_*, constants a0 and a1) in its epilogue.
@@ -590,7 +616,7 @@ extern "C" int tl_gemm_tc_pair_act(const void* X, long long ldx, long long x_row
                                    float a0, float a1, int* status, cudaStream_t stream) {
   TL_REQUIRE(act >= 1 && act <= TL_ACT_LAST, "pair product: activation %d is not one of 1..%d", act, TL_ACT_LAST);
   return pair_product(X, ldx, x_rows, W, ldw, w_rows, 0, bias, C, ldc, M, N, K, 0, out_dtype, nullptr, nullptr, nullptr, nullptr,
-                      0, 0, 1, 1, act, a0, a1, status, stream);
+                      0, 0, 1, 1, act, a0, a1, status, nullptr, nullptr, stream);
 }
 
 // For tests of the bounded waits, as in tc_gemm.cu: the polls after which an mbarrier wait of this file's kernel gives up

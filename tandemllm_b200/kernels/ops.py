@@ -18,7 +18,8 @@ FP32, BF16 = 0, 1
 TL_BAD_ARGUMENT = 100001
 # the gate activations of gated products (TL_ACT_* of csrc/common.cuh) and the router's scoring functions (TL_SCORE_*
 # of csrc/route.cuh), by the names a part's spec gives them
-ACTIVATIONS = {"silu": 1, "gelu": 2, "relu2": 3, "identity": 4, "xielu": 5, "clamped_swish": 6, "softcap": 7, "tanh": 8, "scale": 9}
+ACTIVATIONS = {"silu": 1, "gelu": 2, "relu2": 3, "identity": 4, "xielu": 5, "clamped_swish": 6, "softcap": 7, "tanh": 8, "scale": 9,
+               "gelu_tanh": 10}
 SCORINGS = {"sigmoid": 0, "softmax": 1, "chosen_softmax": 2}
 
 
@@ -65,6 +66,8 @@ _SIGNATURES = {
     "tl_embed_rows": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p],
     "tl_embed_rows_copies": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_float, c_int, c_longlong,
                              c_void_p],
+    "tl_embed_token_pairs": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+                             c_longlong, c_longlong, c_longlong, c_int, c_void_p, c_float, c_void_p],
     "tl_add_rmsnorm_streams": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_void_p,
                                c_int, c_void_p,
                                c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
@@ -83,7 +86,7 @@ _SIGNATURES = {
                      c_int, c_int, c_void_p],
     "tl_gemm_simt_grouped": [c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_longlong, c_longlong, c_void_p,
                              c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                             c_int, c_int, c_void_p],
+                             c_int, c_int, c_void_p, c_void_p, c_void_p],
     "tl_gemm_simt_tile_rows": [],
     "tl_short_conv": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                       c_int, c_int, c_int, c_void_p],
@@ -128,10 +131,10 @@ _SIGNATURES = {
     "tl_gated_group_norm": [c_void_p, c_void_p, c_longlong, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "tl_latent_prepare": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p,
                           c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
-                          c_void_p],
+                          c_int, c_void_p],
     "tl_rmsnorm_rows": [c_void_p, c_longlong, c_void_p, c_float, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p],
     "tl_head_linear": [c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_longlong, c_longlong, c_int, c_int, c_int, c_int,
-                       c_int, c_int, c_void_p, c_longlong, c_void_p],
+                       c_int, c_int, c_void_p, c_longlong, c_int, c_void_p],
     "tl_attention_latent": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_int, c_void_p,
                             c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p],
     "tl_add_layernorm": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int,
@@ -144,7 +147,8 @@ _SIGNATURES = {
                           c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p],
     "tl_recurrence_scan": [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p,
                            c_float, c_float, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int,
-                           c_int, c_int, c_void_p, c_longlong, c_int, c_int, c_float, c_void_p],
+                           c_int, c_int, c_void_p, c_longlong, c_int, c_int, c_float, c_void_p, c_void_p, c_int, c_float,
+                           c_void_p],
     "tl_recurrence_scratch_floats": [c_longlong, c_int, c_int, c_int, c_int],
     "tl_gated_delta_scan": [c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_float,
                             c_float, c_void_p, c_int, c_int, c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_void_p, c_int,
@@ -246,6 +250,20 @@ def embed_rows(table: torch.Tensor, tokens: torch.Tensor, residual: torch.Tensor
           "embed_rows")
 
 
+def embed_token_pairs(table: torch.Tensor, pairs: torch.Tensor, step, last_token: torch.Tensor, residual: torch.Tensor,
+                      status: torch.Tensor, mul_prev: int, mul_cur: int, scale: float = 1.0) -> None:
+    """residual[r] = table[t] * scale + pairs[(before * mul_prev + t * mul_cur) mod buckets] in 32-bit, t the row's token and `before`
+    the one in front of it in its sequence; `pairs` [buckets + 1, hidden], whose last row a sequence's first token reads. `last_token`
+    int32 [slots, 1] holds each request's last token (negative: none yet) and is moved on."""
+    _need(table, None, "embedding table"); _need(pairs, table.dtype, "table of pairs"); _need(residual, torch.float32, "residual")
+    _need(last_token, torch.int32, "last tokens")
+    rows, hidden = residual.shape
+    check(core().tl_embed_token_pairs(ptr(table), ptr(pairs), ptr(step.token_ids), ptr(step.req_of_row), ptr(step.row_start),
+                                      ptr(step.state_slot), ptr(last_token), ptr(residual), rows, hidden, table.shape[0],
+                                      pairs.shape[0] - 1, int(mul_prev), int(mul_cur), dtype_code(table.dtype), ptr(status),
+                                      float(scale), stream()), "embed_token_pairs")
+
+
 class PartialSums:
     """A product's output still in `parts` partial sums [parts, rows, hidden] (32-bit), to be added in order and, when
     `dtype` is given, rounded to it (what the product's own reduction would have stored)."""
@@ -265,8 +283,9 @@ class ExpertRows:
     """A routed expert layer's output still as one row per (row, slot) pair in expert-sorted order [pairs, hidden]
     (32-bit), with what is needed to weigh and add them per row."""
 
-    def __init__(self, rows: torch.Tensor, pos_of_pair: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, parts: int = 1):
-        """`parts` > 1: `rows` is [parts, pairs, hidden], partial sums of a down projection split along k."""
+    def __init__(self, rows: torch.Tensor, pos_of_pair: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor | None, parts: int = 1):
+        """`parts` > 1: `rows` is [parts, pairs, hidden], partial sums of a down projection split along k. `wts` None: the rows
+        are added as they are."""
         self.rows, self.pos_of_pair, self.ids, self.wts, self.parts = rows, pos_of_pair, ids, wts, parts
 
     def materialize(self) -> torch.Tensor:
@@ -385,7 +404,8 @@ def add_rmsnorm(residual: torch.Tensor, delta, weight: torch.Tensor, eps: float,
 
 def add_rmsnorm_pair(residual: torch.Tensor, delta, weight: torch.Tensor, eps: float, out: torch.Tensor, weight2: torch.Tensor | None,
                      out2: torch.Tensor | None, gather: torch.Tensor | None = None, route: dict | None = None) -> torch.Tensor:
-    """residual += delta (None, a branch output in any form, or a `BranchSum` of two); out = weight * row / rms(row) and, with
+    """residual += delta (None, a branch output in any form, or a `BranchSum` of two, one of which may be a `GatedSum` without a
+    gate); out = weight * row / rms(row) and, with
     `weight2`, out2 = weight2 * row / rms(row) of the same new row. `gather` and `route` as in `add_rmsnorm`; the router reads
     the second norm's unrounded rows (the first's without a second)."""
     _need(residual, torch.float32, "residual"); _need(weight, torch.float32, "norm weight"); _need(out, None, "normed")
@@ -394,7 +414,12 @@ def add_rmsnorm_pair(residual: torch.Tensor, delta, weight: torch.Tensor, eps: f
     if weight2 is not None:
         _need(weight2, torch.float32, "norm weight"); _need(out2, out.dtype, "normed")
     dense, experts = [], None
-    for piece in ((delta.first, delta.second) if isinstance(delta, BranchSum) else (delta,)):
+    pieces = [delta.first, delta.second] if isinstance(delta, BranchSum) else [delta]
+    if sum(isinstance(p, GatedSum) and p.gate is None for p in pieces) == 1 and not any(isinstance(p, ExpertRows) for p in pieces):
+        # a dense part beside expert rows: with the other branch's tensor they are just what the kernel adds
+        at = next(i for i, p in enumerate(pieces) if isinstance(p, GatedSum) and p.gate is None)
+        pieces[at:at + 1] = [pieces[at].dense, pieces[at].experts]
+    for piece in pieces:
         if isinstance(piece, ExpertRows) and experts is None:
             experts = piece
         elif isinstance(piece, PartialSums) and piece.dtype is None:
@@ -624,16 +649,17 @@ def gated_group_norm(y: torch.Tensor, z: torch.Tensor, weight, eps: float, group
 
 # ------------------------------------------------------------------------------------------ latent attention
 def latent_prepare(q, kv, c_weight, eps, inv_freq, rot_dims, positions, req_of_row, table, page_size, cache, q_out,
-                   heads: int, dim: int, latent: int, rot_dim: int, status) -> None:
+                   heads: int, dim: int, latent: int, rot_dim: int, status, halves: bool = False) -> None:
     """Writes the normed latent and the rotated shared key part of every row into its page, and every head's rotated query
-    part into `q_out` (float32 [rows, heads, latent + rot_dim]) behind the place of its absorbed part (csrc/attention_latent.cu)."""
+    part into `q_out` (float32 [rows, heads, latent + rot_dim]) behind the place of its absorbed part (csrc/attention_latent.cu).
+    Neighbouring entries are the pairs that turn, or with `halves` entries i and i + rot_dims / 2."""
     _need(q, cache.dtype, "q"); _need(q_out, torch.float32, "q'")
     if kv.dtype != cache.dtype or kv.stride(-1) != 1:
         raise KernelError("latent prepare: the latent's rows in the cache's type with unit stride")
     check(core().tl_latent_prepare(ptr(q), q.stride(0), ptr(kv), kv.stride(0), ptr(c_weight), float(eps), ptr(inv_freq),
                                    int(rot_dims), ptr(positions), ptr(req_of_row), ptr(table), table.shape[1], int(page_size),
                                    cache.shape[0], ptr(cache), ptr(q_out), q.shape[0], heads, dim, latent, rot_dim,
-                                   dtype_code(q.dtype), ptr(status), stream()), "latent_prepare")
+                                   dtype_code(q.dtype), ptr(status), int(halves), stream()), "latent_prepare")
 
 
 def rmsnorm_rows(x: torch.Tensor, n: int, weight: torch.Tensor, eps: float, out: torch.Tensor) -> torch.Tensor:
@@ -648,17 +674,17 @@ def rmsnorm_rows(x: torch.Tensor, n: int, weight: torch.Tensor, eps: float, out:
 
 
 def head_linear(a: torch.Tensor, ld_a: int, a_head: int, w: torch.Tensor, out: torch.Tensor, ld_out: int, out_head: int,
-                rows: int, gate: torch.Tensor | None = None) -> torch.Tensor:
+                rows: int, gate: torch.Tensor | None = None, gate_heads: bool = False) -> torch.Tensor:
     """out[r, h, n] = sum_k a[r, h, k] w[h, n, k] with w [heads, N, K]; `a` and `out` addressed by a row stride and a head
     stride (elements). With `gate` (logits [rows, heads * N] of the operands' type, unit inner stride) the result is
-    multiplied entry by entry by sigmoid(gate)."""
+    multiplied entry by entry by sigmoid(gate); with `gate_heads` the gate is [rows, heads], one logit a head."""
     _need(w, a.dtype, "head weights")
     H, N, K = w.shape
     if gate is not None and (gate.dtype != a.dtype or gate.stride(-1) != 1):
         raise KernelError("head product: a gate of the operands' type with unit stride")
     check(core().tl_head_linear(ptr(a), int(ld_a), int(a_head), ptr(w), ptr(out), int(ld_out), int(out_head), rows, H, N, K,
                                 dtype_code(a.dtype), dtype_code(out.dtype), ptr(gate), gate.stride(0) if gate is not None else 0,
-                                stream()), "head_linear")
+                                int(gate_heads), stream()), "head_linear")
     return out
 
 
@@ -688,16 +714,18 @@ def gemm_simt(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None, out: 
 
 
 def gemm_simt_grouped(a: torch.Tensor, a_gather: torch.Tensor | None, a_div: int, w: torch.Tensor, out: torch.Tensor,
-                      plan: "MoePlan", swiglu: bool | int) -> torch.Tensor:
+                      plan: "MoePlan", swiglu: bool | int, weights: torch.Tensor | None = None) -> torch.Tensor:
     """Per sorted row i of the plan: out[i] = A[row(i)] @ w[expert(i)]^T, with w [E, N(*2 when swiglu), K]. `swiglu`:
-    False for a plain product, True or a code of ACTIVATIONS for act(gate rows) * (up rows), a negated code for act(plain product)."""
+    False for a plain product, True or a code of ACTIVATIONS for act(gate rows) * (up rows), a negated code for act(plain product).
+    `weights` (float32, one number a (row, slot) pair; gated form): the pair's row is multiplied by it in front of the expert."""
     _need(a, w.dtype, "a"); _need(w, None, "w"); _need(out, None, "out")
     E, n_rows_w, K = w.shape
     N = n_rows_w // 2 if int(swiglu) > 0 else n_rows_w
     check(core().tl_gemm_simt_grouped(ptr(a), a.stride(0), ptr(a_gather), a_div, ptr(w), w.stride(1), w.stride(0),
                                       ptr(out), out.stride(0), plan.pairs, N, K, ptr(plan.tile_group),
                                       ptr(plan.tile_row0), ptr(plan.tile_rows), ptr(plan.n_tiles), plan.max_tiles,
-                                      int(swiglu), dtype_code(a.dtype), dtype_code(out.dtype), stream()),
+                                      int(swiglu), dtype_code(a.dtype), dtype_code(out.dtype), ptr(weights),
+                                      ptr(plan.sorted_pairs) if weights is not None else None, stream()),
           "gemm_simt_grouped")
     return out
 
@@ -874,12 +902,13 @@ RECURRENCE_STAGED_ROWS = 8      # a request that brings more rows than this take
 def recurrence_scan(proj, q_col: int, k_col: int, v_col: int, state, state_slot, row_start, requests: int, y, heads: int,
                     key_dim: int, value_dim: int, *, head_decay=None, a_col: int = -1, w=None, w0=None, a_bias=None,
                     rate: float = 0.0, key_eps: float = 0.0, silu_inputs: bool = False, write_state: bool = True,
-                    max_rows: int = 1, q_scale: float = 1.0) -> torch.Tensor:
+                    max_rows: int = 1, q_scale: float = 1.0, turn: tuple | None = None, k_scale: float = 1.0) -> torch.Tensor:
     """The recurrence over a matrix state a head (csrc/recurrence.cu): with `head_decay` (float32 [heads]) the decayed sum of
     outer products, with `w` (float32 [rows, heads * key_dim], the decay's logits) and `a_col` the generalized delta rule,
     with `w` alone the gated outer products (a decay sigmoid(w + w0)^rate a key channel). q is multiplied by `q_scale`. `proj`:
     float32 rows holding q, k, v (and the removal logits at `a_col`) at the given columns; `state` [slots, heads, key_dim,
-    value_dim] float32; `y` [rows, heads * value_dim] float32. `max_rows`: the most rows a request brings; above
+    value_dim] float32; `y` [rows, heads * value_dim] float32. With `head_decay`, `turn` = (positions int32 [rows], inv_freq float32
+    [rot / 2], rot) turns the first `rot` entries of q and k a head (halves layout), and k is multiplied by `k_scale`. `max_rows`: the most rows a request brings; above
     RECURRENCE_STAGED_ROWS the tokens' activations, decays and unit keys are formed side by side first and the scan fetches
     them ahead of its loop."""
     _need(proj, torch.float32, "projections"); _need(state, torch.float32, "state"); _need(y, torch.float32, "y")
@@ -895,7 +924,9 @@ def recurrence_scan(proj, q_col: int, k_col: int, v_col: int, state, state_slot,
                                     w.stride(0) if w is not None else 0, ptr(w0), ptr(a_bias), ptr(head_decay), float(rate),
                                     float(key_eps), int(silu_inputs), ptr(state), state[0].numel(), ptr(state_slot),
                                     ptr(row_start), int(requests), ptr(y), heads, key_dim, value_dim, int(write_state),
-                                    ptr(scratch), rows, sm_count(), rule, float(q_scale), stream()), "recurrence_scan",
+                                    ptr(scratch), rows, sm_count(), rule, float(q_scale), ptr(turn[0]) if turn else None,
+                                    ptr(turn[1]) if turn else None, int(turn[2]) if turn else 0, float(k_scale), stream()),
+          "recurrence_scan",
           kernels=2 if scratch is not None else 1)
     return y
 
@@ -960,14 +991,15 @@ def group_norm_gate(y, gate, ld_gate: int, weight, eps: float, groups: int, scal
                     ) -> torch.Tensor:
     """out = y / rms(y) over each of `groups` equal parts of a row, times `weight`, times sigmoid(gate) (or, with
     `gate_activation` "silu", gate sigmoid(gate)), times `scale`. `gate` begins at the first logit, rows `ld_gate` apart
-    (32-bit or the compute dtype); `out` may be a column slice. A weight of one part's size is shared by all parts."""
+    (32-bit or the compute dtype); `out` may be a column slice. A weight of one part's size is shared by all parts; None: there is
+    none."""
     _need(y, torch.float32, "y")
     rows, width = y.shape
     if out.stride(1) != 1 or out.shape != (rows, width):
         raise KernelError(f"group_norm_gate output of shape {tuple(out.shape)}")
     check(core().tl_group_norm_gate(ptr(y), ptr(gate), int(ld_gate), dtype_code(gate.dtype), ptr(weight), float(eps),
                                     float(scale), ptr(out), out.stride(0), rows, width, int(groups), dtype_code(out.dtype),
-                                    int(gate_activation == "silu"), int(weight.numel() * groups == width and groups > 1),
+                                    int(gate_activation == "silu"), int(weight is not None and weight.numel() * groups == width and groups > 1),
                                     stream()), "group_norm_gate")
     return out
 

@@ -66,11 +66,11 @@ def lib():
         l = load("tensorcore")
         l.tl_gemm_tc.argtypes = [c_void_p, c_longlong, c_longlong, c_void_p, c_longlong, c_longlong, c_longlong, c_void_p,
                                  c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
-                                 c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p]
+                                 c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p]
         l.tl_gemm_tc.restype = c_int
         l.tl_gemm_tc_pair.argtypes = [c_void_p, c_longlong, c_longlong, c_void_p, c_longlong, c_longlong, c_longlong, c_void_p,
                                       c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
-                                      c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p]
+                                      c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p]
         l.tl_gemm_tc_pair.restype = c_int
         l.tl_gemm_tc_pair_act.argtypes = [c_void_p, c_longlong, c_longlong, c_void_p, c_longlong, c_longlong, c_void_p, c_void_p,
                                           c_longlong, c_int, c_int, c_int, c_int, c_int, ctypes.c_float, ctypes.c_float, c_void_p,
@@ -88,7 +88,7 @@ def lib():
                                               c_void_p, c_void_p, c_void_p]
         l.tl_attention_latent_mma.restype = c_int
         l.tl_head_linear_mma.argtypes = [c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_longlong, c_longlong, c_int, c_int,
-                                         c_int, c_int, c_int, c_void_p, c_longlong, c_void_p]
+                                         c_int, c_int, c_int, c_void_p, c_longlong, c_int, c_void_p]
         l.tl_head_linear_mma.restype = c_int
         l.tl_attention_latent_mma_scratch.argtypes = [c_int, c_int, c_int, c_int]
         l.tl_attention_latent_mma_scratch.restype = c_longlong
@@ -136,7 +136,7 @@ def lib():
         l.tl_gemm_skinny_mma.restype = c_int
         l.tl_gemm_skinny_grouped.argtypes = [c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_longlong, c_longlong, c_void_p,
                                              c_longlong, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
-                                             c_int, c_void_p, c_int, c_int, c_void_p, c_void_p]
+                                             c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p]
         l.tl_gemm_skinny_grouped.restype = c_int
         l.tl_gemm_skinny_conv.argtypes = [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p,
                                           c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]
@@ -189,11 +189,11 @@ class TensorCore:
 
     # ---- x @ w^T (+ bias) ----
     def gemm(self, x, w2d, bias, out, *, rows_per_group=0, plan=None, swiglu=False, swap=None, bn=None, n_out=None,
-             defer: bool = False, row_index=None, row_div: int = 1, rows: int | None = None, splits: int = 1):
+             defer: bool = False, row_index=None, row_div: int = 1, rows: int | None = None, splits: int = 1, weights=None):
         """Runs the product into `out`. With `defer`, a product that was split along k is left as partial sums and
         returned as `ops.PartialSums` (nothing is written to `out`); otherwise returns None. With `row_index` (grouped,
         swapped) the plan's position i stands for row row_index[i] // row_div of x, and `rows` is the number of
-        positions."""
+        positions. `weights` (with a plan, gated): a (row, slot) pair's own weight, in front of the activation."""
         M, K = (rows if rows is not None else x.shape[0]), x.shape[1]
         N = n_out if n_out is not None else w2d.shape[0]
         if swap is None:
@@ -215,7 +215,7 @@ class TensorCore:
                                    splits=runs)
                     return ops.PartialSums(partial, runs, M, N, None)
             self.gemm_pair(x, w2d, bias, out, rows_per_group=rows_per_group, plan=plan, gated=int(swiglu), n_out=n_out,
-                           rows=rows)
+                           rows=rows, weights=weights)
             return None
         forced, partial = splits > 1, None
         if forced:
@@ -239,7 +239,7 @@ class TensorCore:
             ops.ptr(bias), out.data_ptr(), out.stride(0), M, N, K, int(swap), bn, int(swiglu), ops.dtype_code(out.dtype),
             ops.ptr(tg), ops.ptr(tr0), ops.ptr(trs), ops.ptr(nt), max_tiles, ops.ptr(row_index), int(row_div), splits,
             ops.ptr(partial), int(not deferred),
-            self.status.data_ptr(), ops.stream())
+            self.status.data_ptr(), ops.ptr(weights), ops.ptr(plan.sorted_pairs) if weights is not None else None, ops.stream())
         _check(code, "gemm_tc", kernels=2 if splits > 1 and not deferred else 1)
         if not deferred or forced:
             return None
@@ -252,12 +252,13 @@ class TensorCore:
         return self._pairs
 
     def gemm_pair(self, x, w2d, bias, out, *, rows_per_group=0, plan=None, gated: int = 0, n_out=None,
-                  rows: int | None = None, per_sm: int | None = None, splits: int = 1) -> None:
+                  rows: int | None = None, per_sm: int | None = None, splits: int = 1, weights=None) -> None:
         """The product on pairs of SMs (csrc/tc_gemm_pair.cu): 256 outputs by up to 256 token rows a pair, the N side
         of its MMAs as many rows as a tile holds. `plan`: tiles of any height up to 256 rows. `per_sm` 2: two CTAs an
         SM, each with half the shared and tensor memory (gated: tiles of up to 128 rows), the form for products bound
         by their weights; default: 2 for a plan with tiles of up to 128 rows, else 1. `splits` > 1: `out` is
-        [splits, M, N] 32-bit and receives the partial results of as many runs of k-blocks (plain product only)."""
+        [splits, M, N] 32-bit and receives the partial results of as many runs of k-blocks (plain product only). A `bias` of
+        the gated form (no plan) holds the gate's numbers, then the up rows'. `weights` (gated, with a plan): as in `gemm`."""
         M, K = (rows if rows is not None else x.shape[0]), x.shape[1]
         N = n_out if n_out is not None else w2d.shape[0]
         tg = tr0 = trs = nt = None
@@ -270,17 +271,20 @@ class TensorCore:
         _check(lib().tl_gemm_tc_pair(x.data_ptr(), x.stride(0), x.shape[0], w2d.data_ptr(), w2d.stride(0), w2d.shape[0],
                                      rows_per_group, ops.ptr(bias), out.data_ptr(), out.stride(0), M, N, K, int(gated),
                                      ops.dtype_code(out.dtype), ops.ptr(tg), ops.ptr(tr0), ops.ptr(trs), ops.ptr(nt),
-                                     max_tiles, plan_rows, per_sm, splits, self.status.data_ptr(), ops.stream()),
+                                     max_tiles, plan_rows, per_sm, splits, self.status.data_ptr(), ops.ptr(weights),
+                                     ops.ptr(plan.sorted_pairs) if weights is not None else None, ops.stream()),
                "gemm_tc_pair")
 
-    def gated(self, x, w_gate_up, out, act: int = 1) -> bool:
-        """out = act(x gate^T) * (x up^T) for w_gate_up = [gate rows; up rows], in the persistent kernel with the gated
+    def gated(self, x, w_gate_up, out, act: int = 1, bias=None) -> bool:
+        """out = act(x gate^T) * (x up^T), each with its half of `bias` [gate; up] where there is one, for w_gate_up = [gate rows; up rows], in the persistent kernel with the gated
         epilogue (`act`: a code of ops.ACTIVATIONS, 1 = SiLU); False (nothing done) for a decode step's few rows or
         operands the kernels do not take."""
         inter = w_gate_up.shape[0] // 2
         if x.shape[0] <= 128 or not usable(x, w_gate_up) or inter % 8 or out.stride(-1) != 1 or out.dtype != torch.bfloat16:
             return False
-        self.gemm(x, w_gate_up, None, out, swiglu=act, swap=False, n_out=inter)
+        if bias is not None and PROMPT_PRODUCT != "pair":
+            return False                        # only the pair product's gated epilogue adds a bias
+        self.gemm(x, w_gate_up, bias, out, swiglu=act, swap=False, n_out=inter)
         return True
 
     def linear(self, x, w, bias, out, defer: bool = False):
@@ -358,10 +362,11 @@ class TensorCore:
             "attention_latent_mma", kernels=2 if n_spans > 1 else 1)
         return True
 
-    def head_linear(self, a, ld_a: int, a_head: int, w, out, ld_out: int, out_head: int, rows: int, gate=None) -> bool:
+    def head_linear(self, a, ld_a: int, a_head: int, w, out, ld_out: int, out_head: int, rows: int, gate=None,
+                    gate_heads: bool = False) -> bool:
         """out[r, h, n] = sum_k a[r, h, k] w[h, n, k] on the tensor cores (csrc/head_linear_mma.cu) for bfloat16 operands
-        (out bfloat16 or float32), times sigmoid(gate[r, h, n]) with `gate` (bfloat16 logits, unit inner stride); False for
-        anything else."""
+        (out bfloat16 or float32), times sigmoid(gate[r, h, n]) (`gate_heads`: gate[r, h]) with `gate` (bfloat16 logits,
+        unit inner stride); False for anything else."""
         if a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or out.dtype not in (torch.bfloat16, torch.float32):
             return False
         if gate is not None and (gate.dtype != torch.bfloat16 or gate.stride(-1) != 1):
@@ -369,7 +374,8 @@ class TensorCore:
         H, N, K = w.shape
         _check(lib().tl_head_linear_mma(a.data_ptr(), int(ld_a), int(a_head), w.data_ptr(), out.data_ptr(), int(ld_out),
                                         int(out_head), rows, H, N, K, ops.dtype_code(out.dtype), ops.ptr(gate),
-                                        gate.stride(0) if gate is not None else 0, ops.stream()), "head_linear_mma")
+                                        gate.stride(0) if gate is not None else 0, int(gate_heads), ops.stream()),
+               "head_linear_mma")
         return True
 
     def in_proj_conv(self, x, w_in, b_in, taps, b_taps, state, state_slot, req_of_row, positions, y,
@@ -420,7 +426,7 @@ class TensorCore:
             # the CTAs with work are the grid's first (up to 32 pairs, see the kernel): 832 -> 881 tok/s at batch 1, even
             # at 16 pairs, 2854 -> 2869 tok/s at 24 pairs, 3434 -> 3388 at 32.
             where = (None, None, None, None, 0, ids.data_ptr(), P, E)
-            gate_up_rows, pos, div = None, self.pair_order(), k
+            gate_up_rows, pos, div, pair_at = None, self.pair_order(), k, None
         else:
             if plan is None or plan.tile_m != 8:
                 plan = part.plan_for(P, x.device, 8).build(ids)
@@ -428,15 +434,17 @@ class TensorCore:
                 part.load.add_(plan.counts)
             where = (plan.tile_group.data_ptr(), plan.tile_row0.data_ptr(), plan.tile_rows.data_ptr(),
                      plan.n_tiles.data_ptr(), plan.max_tiles, None, 0, E)
-            gate_up_rows, pos, div = plan.sorted_pairs.data_ptr(), plan.pos_of_pair, k
+            gate_up_rows, pos, div, pair_at = plan.sorted_pairs.data_ptr(), plan.pos_of_pair, k, plan.sorted_pairs.data_ptr()
+        before = wts if part.weighs_input else None
         _check(lib().tl_gemm_skinny_grouped(x.data_ptr(), x.stride(0), gate_up_rows, div,
                                             part.w_gate_up.data_ptr(), H, I2, act.data_ptr(), inter, inter, H, part.act,
-                                            ops.dtype_code(act.dtype), *where, self.status.data_ptr(), ops.stream()),
+                                            ops.dtype_code(act.dtype), *where, self.status.data_ptr(), ops.ptr(before),
+                                            pair_at if before is not None else None, ops.stream()),
                "gemm_skinny_grouped")
         _check(lib().tl_gemm_skinny_grouped(act.data_ptr(), inter, None, 1, part.w_down.data_ptr(), inter, H, y.data_ptr(), H,
                                             H, inter, 0, ops.dtype_code(y.dtype), *where, self.status.data_ptr(),
-                                            ops.stream()), "gemm_skinny_grouped")
-        return ops.ExpertRows(y, pos, ids, wts)
+                                            None, None, ops.stream()), "gemm_skinny_grouped")
+        return ops.ExpertRows(y, pos, ids, part.output_weights(wts))
 
     def pair_order(self) -> torch.Tensor:
         """0, 1, 2, ...: the places of expert rows that were left in the order of their pairs."""
@@ -475,11 +483,13 @@ class TensorCore:
             part.load.add_(plan.counts)
         act = torch.empty(P, inter, dtype=x.dtype, device=x.device)
         w_gate_up = part.w_gate_up.view(E * I2, H)
+        before = wts if part.weighs_input else None
         if fetch:
             self.gemm(x, w_gate_up, None, act, rows_per_group=I2, plan=plan, swiglu=part.act, swap=True, bn=bn, n_out=inter,
-                      row_index=plan.sorted_pairs, row_div=k, rows=P)
+                      row_index=plan.sorted_pairs, row_div=k, rows=P, weights=before)
         else:
-            self.gemm(xs, w_gate_up, None, act, rows_per_group=I2, plan=plan, swiglu=part.act, swap=swap, bn=bn, n_out=inter)
+            self.gemm(xs, w_gate_up, None, act, rows_per_group=I2, plan=plan, swiglu=part.act, swap=swap, bn=bn, n_out=inter,
+                      weights=before)
         w_down = part.w_down.view(E * H, inter)
         ctas = min(P, E) * -(-H // 128)
         if fetch and ctas < self.sm_count and inter >= 512:
@@ -487,10 +497,10 @@ class TensorCore:
             splits = max(2, min(-(-inter // 64) // 4, -(-self.sm_count // ctas), 16))
             y = self.workspace(splits * P * H)[:splits * P * H].view(splits, P, H)
             self.gemm(act, w_down, None, y[0], rows_per_group=H, plan=plan, swap=True, bn=bn, n_out=H, splits=splits)
-            return ops.ExpertRows(y, plan.pos_of_pair, ids, wts, parts=splits)
+            return ops.ExpertRows(y, plan.pos_of_pair, ids, part.output_weights(wts), parts=splits)
         y = torch.empty(P, H, dtype=torch.float32, device=x.device)
         self.gemm(act, w_down, None, y, rows_per_group=H, plan=plan, swap=swap, bn=bn, n_out=H)
-        return ops.ExpertRows(y, plan.pos_of_pair, ids, wts)
+        return ops.ExpertRows(y, plan.pos_of_pair, ids, part.output_weights(wts))
 
 
     # ---- attention ----

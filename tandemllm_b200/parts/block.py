@@ -19,6 +19,8 @@ that whatever a run order adds to the stream between two layers meets a complete
 
     h = h + (mixer(norm_m(h)) + feed_forward(norm_f(h)))
 
+With one norm for both (`feed_forward_norm` None beside a feed-forward): h = h + (mixer(n) + feed_forward(n)), n = norm_m(h).
+
 Both norms are one kernel behind the adds of what the layer before left (`add_two_norms`), with the router of a routed
 feed-forward inside; what the layer leaves is an `ops.BranchSum`, which the next norm's kernel adds. The feed-forward runs as
 a branch of its own (`Runtime.branch`): its partial sums and the mixer's wait side by side.
@@ -81,7 +83,10 @@ class ParallelResidual:
         if getattr(ff, "absent", False):
             return layer.mixer.forward(layer.mixer_norm.add_norm(residual, pending), step, cache, writes_cache=writes_cache)
         route = ff.router_args(residual.shape[0], residual.device) if hasattr(ff, "router_args") else None
-        n, nf = layer.mixer_norm.add_two_norms(residual, pending, layer.feed_forward_norm, route)
+        if layer.feed_forward_norm is None:
+            n = nf = layer.mixer_norm.add_norm(residual, pending, route=route)
+        else:
+            n, nf = layer.mixer_norm.add_two_norms(residual, pending, layer.feed_forward_norm, route)
         with ff.runtime.branch(1):
             out = ff.forward(nf, step, routing=(route["ids"], route["wts"])) if route is not None else ff.forward(nf, step)
         return ops.BranchSum(layer.mixer.forward(n, step, cache, writes_cache=writes_cache), out)

@@ -7,9 +7,13 @@
                                                                          ref.py:185-214
 
 With `gated: False` an expert has no gate matrix: expert(n) = down( act(up n) ), the activation in the up product's epilogue.
+With `weigh: input` the weight multiplies the row in front of the expert instead of what the expert makes of it: out = sum of
+expert(w n); it meets the gate's and the up product's 32-bit sums in front of the activation, and the rows are added as they are.
 With the scoring `chosen_softmax` the bias is part of the logits, and the weights are the softmax over the chosen experts' logits.
 
-The gate's activation (`activation`: silu, gelu, relu2, identity) and the router's scoring function (`scoring`:
+The dense form may have biases (`biases`: their tensors' names): out = down( act(gate n + b_g) * (up n + b_u) ) + b_d.
+
+The gate's activation (`activation`: silu, gelu, gelu_tanh, relu2, identity) and the router's scoring function (`scoring`:
 sigmoid, or softmax over all experts) are parameters of the parts' specs, passed to the kernels as codes; LFM2 uses
 silu and sigmoid, and another architecture's gated or routed feed-forward reuses the same fused kernels by naming its own.
 
@@ -49,11 +53,16 @@ class SwiGLU(Part):
         self.gate_constants = gate_constants_of(spec)
         self.suffix = str(spec.get("weight_suffix", ".weight"))
         self.n = {k: prefix + v for k, v in spec["names"].items()}
+        self.bias_names = {k: prefix + v for k, v in (spec.get("biases") or {}).items()}
+        if self.bias_names and set(self.bias_names) != {"gate", "up", "down"}:
+            raise ValueError(f"biases of {sorted(self.bias_names)}: the gate, the up and the down product have one each, or none has")
+        self.b_gate_up = self.b_down = None
 
     def weight_specs(self, present=None):
         H, I, sfx = self.hidden_size, self.inter, self.suffix
         return [TensorSpec(self.n["gate"] + sfx, (I, H)), TensorSpec(self.n["up"] + sfx, (I, H)),
-                TensorSpec(self.n["down"] + sfx, (H, I))]
+                TensorSpec(self.n["down"] + sfx, (H, I))] + \
+               [TensorSpec(name, (H if k == "down" else I,), "vector", "bias") for k, name in self.bias_names.items()]
 
     def bind(self, read, runtime):
         self.runtime = runtime
@@ -61,16 +70,20 @@ class SwiGLU(Part):
         self.w_gate_up = torch.cat([runtime.matrix(read(self.n["gate"] + sfx)),
                                     runtime.matrix(read(self.n["up"] + sfx))]).contiguous()
         self.w_down = runtime.matrix(read(self.n["down"] + sfx))
+        if self.bias_names:
+            b = {k: runtime.vector(read(name)) for k, name in self.bias_names.items()}
+            self.b_gate_up, self.b_down = torch.cat([b["gate"], b["up"]]).contiguous(), b["down"]
 
     def forward(self, x, step):
         act = torch.empty(x.shape[0], self.inter, dtype=x.dtype, device=x.device)
         tc = self.runtime.tensorcore
         if self.gate_constants is not None:
             ops.gate_constants(*self.gate_constants)
-        if tc is None or not tc.gated(x, self.w_gate_up, act, self.act):      # prompts: gate, up and act(gate) * up in one kernel
-            gu = linear(self.runtime, x, self.w_gate_up)
+        # prompts: gate, up and act(gate) * up in one kernel
+        if tc is None or not tc.gated(x, self.w_gate_up, act, self.act, self.b_gate_up):
+            gu = linear(self.runtime, x, self.w_gate_up, self.b_gate_up)
             ops.gated_mul(gu, act, self.act)
-        return linear(self.runtime, act, self.w_down, out_dtype=torch.float32, defer=True)
+        return linear(self.runtime, act, self.w_down, self.b_down, out_dtype=torch.float32, defer=True)
 
 
 @register_part("feed_forward", "dense_act")
@@ -154,6 +167,10 @@ class SigmoidTopKExperts(Part):
             if self.act > ops.ACTIVATIONS["identity"]:
                 raise ValueError(f"ungated experts with the activation {spec.get('activation')!r}: silu, gelu, relu2 or identity")
             self.act = -self.act            # how the grouped products are asked for the ungated form
+        weigh = str(spec.get("weigh", "output"))
+        if weigh not in ("input", "output") or (weigh == "input" and not self.gated):
+            raise ValueError(f"experts weighed at their {weigh!r}: output, or for gated experts input")
+        self.weighs_input = weigh == "input"
         self.suffix = str(spec.get("weight_suffix", ".weight"))
         self.sep = str(spec.get("expert_separator", "."))       # between the experts' common name and an expert's number
         if not 0 < self.top_k <= self.num_experts:
@@ -253,6 +270,10 @@ class SigmoidTopKExperts(Part):
                         self.scoring, self.groups)
         return ids, wts
 
+    def output_weights(self, wts):
+        """What the expert rows are weighed by when they are added (None: as they are, the weights stood in front)."""
+        return None if self.weighs_input else wts
+
     def plan_for(self, pairs: int, device, tile_rows: int | None = None) -> ops.MoePlan:
         """The routing-plan buffers for up to `pairs` pairs and token tiles of `tile_rows` rows (kept and reused)."""
         tile_rows = tile_rows or ops.simt_tile_rows()
@@ -283,10 +304,11 @@ class SigmoidTopKExperts(Part):
         if self.load is not None:
             self.load.add_(plan.counts)
         act = torch.empty(R * self.top_k, self.inter, dtype=x.dtype, device=x.device)
-        ops.gemm_simt_grouped(x, plan.sorted_pairs, self.top_k, self.w_gate_up, act, plan, swiglu=self.act)
+        ops.gemm_simt_grouped(x, plan.sorted_pairs, self.top_k, self.w_gate_up, act, plan, swiglu=self.act,
+                              weights=wts if self.weighs_input else None)
         y = torch.empty(R * self.top_k, H, dtype=torch.float32, device=x.device)
         ops.gemm_simt_grouped(act, None, 1, self.w_down, y, plan, swiglu=False)
-        return ops.ExpertRows(y, plan.pos_of_pair, ids, wts)
+        return ops.ExpertRows(y, plan.pos_of_pair, ids, self.output_weights(wts))
 
 
 @register_part("feed_forward", "shared_and_routed")
@@ -345,7 +367,8 @@ class SharedAndRouted(Part):
 
     def forward(self, x, step, routing=None):
         routed = self.routed.forward(x, step, routing=routing)
-        shared = self.shared.forward(x, step)
+        with self.runtime.branch(4):        # the routed part's rows may still be partial sums, as this part's output may
+            shared = self.shared.forward(x, step)
         gate = None
         if self.w_gate is not None:
             gate = ops.row_dot(x, self.w_gate, torch.empty(x.shape[0], 1, dtype=torch.float32, device=x.device))

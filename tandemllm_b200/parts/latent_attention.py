@@ -6,9 +6,11 @@
   softmax over the visible keys (0 <= i - j < window, or all); out = o(concatenated heads)
   with a `sink` tensor named ([heads]): a head's softmax denominator also holds exp(sink_h), which has no key and no value, is
   not scaled and counts once; with a `gate` matrix named ([heads * value_dim, hidden]): the concatenated heads are multiplied
-  entry by entry by sigmoid(gate n), n the mixer's input, before the out projection
+  entry by entry by sigmoid(gate n), n the mixer's input, before the out projection; with `gate_heads` the matrix is [heads, hidden]
+  and head h's whole output is multiplied by sigmoid(gate n)_h
 
-The position encoding is a part of its own (a kind with `fused_rotary_pairs()`); it turns the rotated parts only. What is
+The position encoding is a part of its own (a kind with `fused_rotary_pairs()`, neighbouring entries, or `fused_rotary()`, the two
+halves); it turns the rotated parts only. What is
 stored a token is c and rot(k_r): one row of kv_rank + rot_dim numbers (`PagedNeed(1, kv_rank + rot_dim, window,
 values=False)`). The products with uk and uv are regrouped so that no key or value of a head is ever formed (csrc/
 attention_latent.cu): q'_h = uk_h^T q_unrotated, scores against the cached rows, the weighted sum of the latents, then uv_h.
@@ -46,13 +48,17 @@ class LatentAttentionMixer(Part):
         self.position = make_part("position_encoding", spec["position"], head_dim=self.rot_dim)
         self.n = {k: prefix + v for k, v in spec["names"].items()}
         self.has_sink, self.has_gate = "sink" in self.n, "gate" in self.n
+        self.gate_heads = bool(spec.get("gate_heads", False))
+        self.halves = not hasattr(self.position, "fused_rotary_pairs")
+        if getattr(self.position, "magnitude", 1.0) != 1.0:
+            raise ValueError("latent attention turns with plain sines and cosines: no magnitude on them")
         self.sinks = None
 
     def weight_specs(self, present=None):
         n, W, H = self.n, self.hidden_size, self.heads
         more = [TensorSpec(n["sink"], (H,), "vector", "bias")] if self.has_sink else []
         if self.has_gate:
-            more.append(TensorSpec(n["gate"], (H * self.vdim, W)))
+            more.append(TensorSpec(n["gate"], (H if self.gate_heads else H * self.vdim, W)))
         return more + [TensorSpec(n["dq"], (self.q_rank, W)), TensorSpec(n["dq_norm"], (self.q_rank,), "vector", "ones"),
                 TensorSpec(n["uq"], (H * (self.dim + self.rot_dim), self.q_rank)),
                 TensorSpec(n["dkv"], (self.kv_rank + self.rot_dim, W)),
@@ -102,10 +108,10 @@ class LatentAttentionMixer(Part):
         kv = down[:, self.kv_at:self.kv_at + Dk]
         gate = down[:, self.gate_at:] if self.has_gate else None
         table = step.block_tables[cache.group]
-        inv_freq, rot_dims = self.position.fused_rotary_pairs()
+        inv_freq, rot_dims = self.position.fused_rotary() if self.halves else self.position.fused_rotary_pairs()
         qa = torch.empty(R, H, Dk, dtype=torch.float32, device=dev)
         ops.latent_prepare(q, kv, self.w_dkv_norm, self.eps, inv_freq, rot_dims, step.positions, step.req_of_row, table,
-                           cache.page_size, cache.k, qa, H, D, L, Rr, rt.status)
+                           cache.page_size, cache.k, qa, H, D, L, Rr, rt.status, self.halves)
         fast = rt.attention_kernels
         if D > 0 and (fast is None or not fast.head_linear(q, q.stride(0), D + Rr, self.w_uk_t, qa, H * Dk, Dk, R)):
             ops.head_linear(q, q.stride(0), D + Rr, self.w_uk_t, qa, H * Dk, Dk, R)
@@ -114,6 +120,6 @@ class LatentAttentionMixer(Part):
             ops.attention_latent(qa, cache.k, table, cache.page_size, step.req_of_row, step.positions, self.scale, self.window,
                                  ol, L, rt.status, self.sinks)
         o = torch.empty(R, H * self.vdim, dtype=dt, device=dev)
-        if fast is None or not fast.head_linear(ol, H * L, L, self.w_uv, o, H * self.vdim, self.vdim, R, gate):
-            ops.head_linear(ol, H * L, L, self.w_uv, o, H * self.vdim, self.vdim, R, gate)
+        if fast is None or not fast.head_linear(ol, H * L, L, self.w_uv, o, H * self.vdim, self.vdim, R, gate, self.gate_heads):
+            ops.head_linear(ol, H * L, L, self.w_uv, o, H * self.vdim, self.vdim, R, gate, self.gate_heads)
         return linear(rt, o, self.w_out, out_dtype=torch.float32, defer=True)

@@ -4,6 +4,9 @@ mixer that runs several mixers side by side on the same rows.
 `decayed_linear_attention`: q = act(W_q n), k = act(W_k n) (heads x head_dim), v = act(W_v n) (heads x value_dim);
     a head: S <- c_h S + k v^T, o = S^T q with the new S, c_h a fixed number a head (`decay`); the concatenated heads are
     brought to unit root mean square together, times the weight `norm`, times sigmoid(W_g n), and projected by W_o.
+    Options: a `position` encoding (the two halves of a head's first entries turn) on q and k, a factor `key_scale` on k behind it,
+    `norm_each`: every head's o is brought to unit root mean square on its own (without `norm` among the names there is no weight),
+    `gate_activation` silu in the place of the sigmoid.
 
 `delta_rule`: r, k, v = W_r n, W_k n, W_v n (heads x head_dim each). A decay a key channel d = exp(-decay_rate *
     sigmoid(W_w2 tanh(W_w1 n) + w0)), a removal rate a key channel a = sigmoid(W_a n + a_b), the unit key
@@ -60,6 +63,16 @@ class DecayedLinearAttention(Part):
         self.activation = str(spec.get("activation", "silu"))
         if self.activation not in ("silu", "identity"):
             raise ValueError(f"activation {self.activation!r} on q, k, v: silu or identity")
+        self.position = make_part("position_encoding", spec["position"], head_dim=self.head_dim) if spec.get("position") else None
+        if self.position is not None and (hasattr(self.position, "fused_rotary_pairs") or self.activation != "identity"
+                                          or getattr(self.position, "magnitude", 1.0) != 1.0):
+            raise ValueError("a position encoding on a recurrence's q and k: the two halves of a head turn, without an activation")
+        self.key_scale = float(spec.get("key_scale", 1.0))
+        self.norm_groups = self.heads if spec.get("norm_each", False) else 1
+        self.gate_activation = str(spec.get("gate_activation", "sigmoid"))
+        if self.gate_activation not in ("sigmoid", "silu"):
+            raise ValueError(f"gate activation {self.gate_activation!r}: sigmoid or silu")
+        self.w_norm = None
         self.eps = float(spec["eps"])
         self.n = {k: prefix + v for k, v in spec["names"].items()}
 
@@ -70,14 +83,17 @@ class DecayedLinearAttention(Part):
     def weight_specs(self, present=None):
         n, W, H, D, VD = self.n, self.hidden_size, self.heads, self.head_dim, self.value_dim
         return [TensorSpec(n["q"], (H * D, W)), TensorSpec(n["k"], (H * D, W)), TensorSpec(n["v"], (H * VD, W)),
-                TensorSpec(n["gate"], (H * VD, W)), TensorSpec(n["norm"], (H * VD,), "vector", "ones"),
-                TensorSpec(n["out"], (W, H * VD))]
+                TensorSpec(n["gate"], (H * VD, W)), TensorSpec(n["out"], (W, H * VD))] + \
+               ([TensorSpec(n["norm"], (H * VD,), "vector", "ones")] if "norm" in n else [])
 
     def bind(self, read, runtime):
         self.runtime = runtime
         n = self.n
         self.w_in, self.col = _stack([(x, runtime.matrix(read(n[x]))) for x in ("q", "k", "v", "gate")])
-        self.w_norm = runtime.vector(read(n["norm"]))
+        if "norm" in n:
+            self.w_norm = runtime.vector(read(n["norm"]))
+        if self.position is not None:
+            self.position.bind(read, runtime)
         self.w_out = runtime.matrix(read(n["out"]))
         self.head_decay = torch.tensor(self.decay, dtype=torch.float64).to(torch.float32).to(runtime.device)
 
@@ -88,11 +104,16 @@ class DecayedLinearAttention(Part):
         R, dev = x.shape[0], x.device
         proj = linear(self.runtime, x, self.w_in, out_dtype=torch.float32)
         y = torch.empty(R, self.out_dim, dtype=torch.float32, device=dev)
+        turn = None
+        if self.position is not None:
+            inv_freq, rot = self.position.fused_rotary()
+            turn = (step.positions, inv_freq, rot) if rot else None
         ops.recurrence_scan(proj, self.col["q"], self.col["k"], self.col["v"], cache.state, step.state_slot, step.row_start,
                             step.n_requests, y, self.heads, self.head_dim, self.value_dim, head_decay=self.head_decay,
                             silu_inputs=self.activation == "silu", write_state=writes_cache,
-                            max_rows=step.max_rows_per_request)
-        return ops.group_norm_gate(y, proj[:, self.col["gate"]:], proj.stride(0), self.w_norm, self.eps, 1, out_scale, out)
+                            max_rows=step.max_rows_per_request, turn=turn, k_scale=self.key_scale)
+        return ops.group_norm_gate(y, proj[:, self.col["gate"]:], proj.stride(0), self.w_norm, self.eps, self.norm_groups, out_scale,
+                                   out, gate_activation=self.gate_activation)
 
     def forward(self, x, step, cache, writes_cache: bool = True):
         o = torch.empty(x.shape[0], self.out_dim, dtype=x.dtype, device=x.device)

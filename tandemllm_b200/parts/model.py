@@ -2,12 +2,13 @@
 
   h = embed[tokens] (times the spec's embedding scale); for each site of the schedule: run its layer on its cache; h = final_norm(h);
   logits = h @ head^T in 32-bit, head = the embedding when tied   (engine/models/lfm2_moe/ref.py:218-241)
+  with `token_pairs` in the spec the embedded row is the sum of two: the token's own and the one of (token before, token)
   with a soft cap c in the spec: logits <- c tanh(logits / c); with a logit scale: logits <- logits * scale
   with `streams` in the spec the residual is [streams, rows, hidden], every stream starts as the embedded row, the layers'
   arrangement rewrites them, and the last norm reads their sum
 
-The model owns no cache: `cache_needs()` tells the cache manager what every site needs and `forward` is
-given the per-site caches it made. It computes the final norm and the head for the wanted rows only.
+The model owns no cache: `cache_needs()` tells the cache manager what every site needs (and, behind the sites, what the embedding
+does: a request's last token) and `forward` is given the per-site caches it made. It computes the final norm and the head for the wanted rows only.
 """
 
 from __future__ import annotations
@@ -18,7 +19,7 @@ from ..config.spec import ModelSpec
 from ..kernels import ops
 from ..settings import SETTINGS
 from ..weights.loader import TensorSpec
-from .base import Runtime, StepContext, make_part
+from .base import Runtime, SlotNeed, StepContext, make_part
 from .block import Layer
 from .linear import linear
 
@@ -30,12 +31,14 @@ class DecoderModel:
         self.layers = [Layer(ls, spec.hidden_size) for ls in spec.layers]
         self.final_norm = make_part("norm", spec.final_norm, prefix=spec.final_norm_prefix, size=spec.hidden_size)
         self.runtime: Runtime | None = None
-        self.embedding = self.head = None
+        self.embedding = self.head = self.pair_embedding = None
 
     # ---- weights ----
     def weight_specs(self, present: set[str] | None = None) -> list[TensorSpec]:
         s = self.spec
         out = [TensorSpec(s.embedding_name, (s.vocab_size, s.hidden_size))]
+        if s.token_pairs:
+            out.append(TensorSpec(s.token_pairs.tensor, (s.token_pairs.buckets + 1, s.hidden_size)))
         out += self.final_norm.weight_specs(present)
         if s.head_name:
             out.append(TensorSpec(s.head_name, (s.vocab_size, s.hidden_size)))
@@ -61,6 +64,8 @@ class DecoderModel:
         weights.check(specs, ignore=(lambda n: n in ignored) if ignored else None)
         self.runtime = runtime
         self.embedding = runtime.matrix(weights.read(s.embedding_name))
+        if s.token_pairs:
+            self.pair_embedding = runtime.matrix(weights.read(s.token_pairs.tensor))
         self.head = runtime.matrix(weights.read(s.head_name)) if s.head_name else self.embedding
         self.final_norm.bind(weights.read, runtime)
         for layer in self.layers:
@@ -107,7 +112,7 @@ class DecoderModel:
                     dense += part.step_bytes(elem)
         dense += self.final_norm.step_bytes(elem)
         head = self.vocab_size * self.hidden_size * elem
-        embed = batch * self.hidden_size * elem
+        embed = batch * self.hidden_size * elem * (2 if self.spec.token_pairs else 1)
         return {"dense": dense, "experts": experts, "head": head, "embedding_rows": embed,
                 "total": dense + experts + head + embed}
 
@@ -119,16 +124,25 @@ class DecoderModel:
 
     # ---- caches ----
     def cache_needs(self) -> list:
-        """Per site of the schedule: the need of its mixer, or None when the site reads another site's cache."""
-        return [None if site.cache_of is not None else self.layers[site.layer].mixer.cache_need()
-                for site in self.spec.schedule]
+        """Per site of the schedule: the need of its mixer, or None when the site reads another site's cache; last, with a table of
+        token pairs, the embedding's: a request's last token (-1: it has none yet)."""
+        needs = [None if site.cache_of is not None else self.layers[site.layer].mixer.cache_need()
+                 for site in self.spec.schedule]
+        return needs + [SlotNeed((1,), torch.int32, init=-1)] if self.spec.token_pairs else needs
 
     # ---- the forward pass of one batch ----
     def forward(self, step: StepContext, site_caches: list) -> torch.Tensor:
         rt = self.runtime
         shape = (step.n_rows, self.hidden_size)
         residual = torch.empty((self.spec.streams,) + shape if self.spec.streams else shape, dtype=torch.float32, device=rt.device)
-        ops.embed_rows(self.embedding, step.token_ids, residual, rt.status, self.spec.embedding_scale)
+        pairs = self.spec.token_pairs
+        if pairs is None:
+            ops.embed_rows(self.embedding, step.token_ids, residual, rt.status, self.spec.embedding_scale)
+        else:
+            if self.spec.streams:
+                raise NotImplementedError("a second embedding over a residual of several streams")
+            ops.embed_token_pairs(self.embedding, self.pair_embedding, step, site_caches[len(self.spec.schedule)].state, residual,
+                                  rt.status, pairs.mul_prev, pairs.mul_cur, self.spec.embedding_scale)
         pending = None
         ranges = SETTINGS.is_set("NVTX")             # named ranges for profilers: the step, and each layer in run order
         if ranges:
