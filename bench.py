@@ -23,6 +23,8 @@ requests at a context of 8192 tokens. A "step" is one decode step of the whole b
 feed-forwards.
 `--design niralix` does the same for Niralix beside an LFM2 MoE model of short-convolution and attention layers.
 `--design gifopel` does the same for Gifopel beside a Sebilorn model (matrix states and attention, dense) and an LFM2 MoE model.
+`--design dipivik` does the same for Dipivik beside a Puripel model (latent attention and state spaces, routed experts) and a Sebilorn
+model (decayed linear attention and attention, dense).
 `--design sifupel` measures the Sifupel design beside the closest existing model (an LFM2 configuration of attention layers
 and dense feed-forwards only) at a few equal layer sizes: prefill and decode throughput, and every launch summed by kernel
 family with its fraction of the measured peak (its own line; the default workload and line are untouched).
@@ -361,6 +363,7 @@ class LaunchTimer:
         return {"tl_gemm_skinny_mma": "dense products (register-only)", "tl_gemm_skinny_conv": "in-projection + short conv",
                 "tl_add_rmsnorm": "residual add + norm (+ router, + deferred sums)",
                 "tl_add_rmsnorm_streams": "residual add + norm (+ router, + deferred sums)", "tl_embed_rows_copies": "embedding",
+                "tl_embed_token_pairs": "embedding",
                 "tl_paged_attention_mma": "attention", "tl_paged_attention_tc": "attention",
                 "tl_paged_attention_split": "attention", "tl_paged_attention_simt": "attention",
                 "tl_attention_join": "attention join", "tl_qk_prepare": "q/k norm + rotary + cache write",
@@ -1268,6 +1271,94 @@ def gifopel_compare(a) -> int:
     return 0
 
 
+DIPIVIK_SIZES = {
+    "1k": dict(width=1024, layers=8, vocab=32768, buckets=65537, heads=16, dim=64, rot=32, vdim=64, kv_rank=256, q_rank=512, window=1024,
+               r_heads=16, r_dim=64, r_vdim=64, ff=2816, experts=32, top=4, expert_ff=512, shared=1024),
+    "2k": dict(width=2048, layers=12, vocab=65536, buckets=131071, heads=32, dim=128, rot=64, vdim=128, kv_rank=512, q_rank=1024,
+               window=2048, r_heads=16, r_dim=128, r_vdim=128, ff=5632, experts=64, top=6, expert_ff=768, shared=1536),
+}
+
+
+def dipivik_compare(a) -> int:
+    """Dipivik beside its closest existing models at equal width, depth, vocabulary, heads and state sizes: a Puripel model (the same
+    latent attention, a state-space layer with as large a state where Dipivik has retention, routed experts of the same size with a
+    shared one in every layer) and a Sebilorn model (decayed linear attention where Dipivik has retention, windowed attention with
+    as many heads where it has latent attention, dense feed-forwards). Dipivik's layers repeat: latent attention + experts, retention
+    + dense, latent attention + dense, retention + experts. Work: latent attention 2 (kv_rank + rot_dim) + 2 kv_rank flops a visible
+    (row, key, head) and, decoding, the bytes of the visible cached rows; the heads' products; a recurrence 6 flops a (row, head,
+    key, value) on the CUDA cores and, decoding, the states read and written; the norms the 32-bit rows in and out."""
+    from tandemllm_b200.config import DipivikConfig, PuripelConfig, SebilornConfig
+    pk = peaks()
+    tokens, batch = a.prefill_tokens, a.batch
+    elem = 2 if a.dtype == "bfloat16" else 4
+    out = []
+    for label in (a.design_sizes.split(",") if a.design_sizes else DIPIVIK_SIZES):
+        z = DIPIVIK_SIZES[label]
+        W, L, V, context = z["width"], z["layers"], z["vocab"], z["window"]
+        RH, RD, RV = z["r_heads"], z["r_dim"], z["r_vdim"]
+        dense = {"kind": "dense", "ff": z["ff"]}
+        moe = {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"]}, "expert": {"ff": z["expert_ff"]},
+               "shared": {"ff": z["shared"]}}
+        latent = {"heads": z["heads"], "dim": z["dim"], "rot_dim": z["rot"], "vdim": z["vdim"], "kv_rank": z["kv_rank"],
+                  "q_rank": z["q_rank"], "scale": (z["dim"] + z["rot"]) ** -0.5, "rot": {"base": 10000.0, "dims": z["rot"]},
+                  "mask": {"size": z["window"]}}
+        decay = [1.0 - 2.0 ** (-3 - 5 * h / max(RH - 1, 1)) for h in range(RH)]
+        ret = {"heads": RH, "dim": RD, "vdim": RV, "decay": decay, "rot": {"base": 1e6, "dims": RD}}
+        cycle = [("latent_attention", latent, moe), ("retention", ret, dense), ("latent_attention", latent, dense), ("retention", ret, moe)]
+        dip = DipivikConfig.from_dict({
+            "architecture": "Dipivik", "vocab": V, "width": W, "norm": {"eps": 1e-6}, "logit_softcap": 20.0,
+            "embedding": {"bigram": {"buckets": z["buckets"], "mul_prev": 31, "mul_cur": 17}},
+            "layers": [dict(zip(("type", "mixer", "mlp"), cycle[i % 4])) for i in range(L)]})
+        pmoe = {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"], "scale": 1.0},
+                "expert": {"ff": z["expert_ff"], "limit": 7.0}, "shared": {"ff": z["shared"], "limit": 7.0}}
+        ssm = {"heads": RH, "vdim": RV, "state": RD, "groups": RH, "conv": 4, "norm_groups": RH}
+        pur = PuripelConfig.from_dict({"architecture": "Puripel", "vocab": V, "width": W, "norm": {"eps": 1e-6}, "layers": [
+            {"type": "latent_attention", "mixer": latent, "mlp": pmoe} if i % 2 == 0 else {"type": "mamba2", "mixer": ssm, "mlp": pmoe}
+            for i in range(L)]})
+        nd = 64 if z["dim"] + z["rot"] <= 96 else 128
+        att = {"heads": z["heads"], "kv_heads": max(1, z["heads"] // 4), "dim": nd, "vdim": nd, "scale": nd ** -0.5,
+               "rot": {"base": 1e6, "dims": nd}, "mask": {"size": z["window"]}}
+        seb = SebilornConfig.from_dict({"architecture": "Sebilorn", "vocab": V, "width": W, "norm": {"eps": 1e-6}, "logit_softcap": 20.0,
+                                        "embedding": {"scale": 1.0}, "layers": [
+            {"type": "attention", "mixer": att, "mlp": dense} if i % 2 == 0 else
+            {"type": "lightning", "mixer": {"heads": RH, "dim": RD, "vdim": RV, "decay": decay}, "mlp": dense} for i in range(L)]})
+        n_att, n_ret = (L + 1) // 2, L // 2
+        pairs = sum(min(i + 1, z["window"]) for i in range(tokens))
+        H, Lr, Dk = z["heads"], z["kv_rank"], z["kv_rank"] + z["rot"]
+        state = float(RH * RD * RV)
+        row = {"sizes": dict(z, label=label), "prefill_tokens": tokens, "batch": batch, "context": context}
+        for name, cfg in (("dipivik", dip), ("puripel", pur), ("sebilorn", seb)):
+            entry = time_design(a, cfg, context)
+            recurrence = (6.0 * tokens * state * n_ret, 8.0 * batch * state * n_ret)
+            work = {"latent attention": (pairs * H * (2.0 * Dk + 2.0 * Lr) * n_att, float(elem) * batch * context * Dk * n_att),
+                    "products a head": (2.0 * tokens * H * Lr * (z["dim"] + z["vdim"]) * n_att,
+                                        float(elem) * H * Lr * (z["dim"] + z["vdim"]) * n_att),
+                    "attention": (4.0 * nd * H * pairs * n_att, 2.0 * elem * batch * att["kv_heads"] * nd * context * n_att),
+                    "matrix-state recurrence": recurrence, "state-space recurrence": recurrence}
+            # one norm a layer: the row in and out, two branches in, a normed row out; a norm a sublayer: a branch in, a normed row out
+            norm_bytes = W * ((4.0 * 4 + elem) * L if name == "dipivik" else (4.0 * 3 + elem) * (2 * L + 1))
+            for table, rows_ in ((entry["prefill"]["families"], tokens), (entry["decode"]["families"], batch)):
+                for fam in ("residual add + norm (+ router, + deferred sums)", "residual add + layer norm"):
+                    if fam in table and name != "puripel":      # (Puripel's norms behind its branches are a family of their own)
+                        rate = norm_bytes * rows_ / table[fam]["ms"] / 1e6
+                        table[fam].update(GBps_rows_only=round(rate, 1), frac_hbm_rows_only=round(rate / pk["hbm_gbs"], 4))
+            for fam, (flops, nbytes) in work.items():
+                pre, dec = entry["prefill"]["families"].get(fam), entry["decode"]["families"].get(fam)
+                if pre:
+                    pre["TFLOPs"] = round(flops / pre["ms"] / 1e9, 2)
+                    if "recurrence" not in fam and a.dtype == "bfloat16":
+                        pre["frac_of_measured_bf16"] = round(flops / pre["ms"] / 1e9 / pk["bf16_tflops"], 4)
+                if dec:
+                    dec["GBps"] = round(nbytes / dec["ms"] / 1e6, 1)
+                    dec["frac_hbm"] = round(nbytes / dec["ms"] / 1e6 / pk["hbm_gbs"], 4)
+            row[name] = entry
+        out.append(row)
+    print(json.dumps({"design_compare": "dipivik beside puripel (latent attention and state spaces, routed experts) and sebilorn (decayed "
+                                        "linear attention and attention, dense)", "dtype": a.dtype, "peaks": pk,
+                      "data": "synthetic: random weights, uniform random token ids, random cached rows as context", "rows": out}))
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1302,18 +1393,19 @@ def main() -> int:
                     help="programmatic dependent launch between the kernels (for comparison; ordinary launches by default)")
     ap.add_argument("--profile", action="store_true",
                     help="bracket the timed decode steps with cudaProfilerStart/Stop (for ncu --profile-from-start off)")
-    ap.add_argument("--design", choices=("sifupel", "puripel", "sebilorn", "niralix", "gifopel"),
+    ap.add_argument("--design", choices=("sifupel", "puripel", "sebilorn", "niralix", "gifopel", "dipivik"),
                     help="measure this design beside the closest existing model at equal layer sizes (its own line)")
     ap.add_argument("--design-sizes", default="", help="--design: which of " + ", ".join(DESIGN_SIZES) + " (sifupel) or "
                     + ", ".join(PURIPEL_SIZES) + " (puripel) or " + ", ".join(SEBILORN_SIZES) + " (sebilorn) or " + ", ".join(NIRALIX_SIZES)
-                    + " (niralix) or " + ", ".join(GIFOPEL_SIZES) + " (gifopel) (default: all)")
+                    + " (niralix) or " + ", ".join(GIFOPEL_SIZES) + " (gifopel) or " + ", ".join(DIPIVIK_SIZES)
+                    + " (dipivik) (default: all)")
     a = ap.parse_args()
     if a.impl == "reference":
         return reference_arm(a)
     if a.design:
         a.warmup = max(a.warmup, 3)
         return {"puripel": puripel_compare, "sebilorn": sebilorn_compare, "niralix": niralix_compare,
-                "gifopel": gifopel_compare}.get(a.design, design_compare)(a)
+                "gifopel": gifopel_compare, "dipivik": dipivik_compare}.get(a.design, design_compare)(a)
     if a.gpus != 1:
         print(json.dumps({"error": f"this engine runs on one GPU; --gpus {a.gpus} is not implemented", "n_gpus": a.gpus}))
         return 2
