@@ -159,8 +159,12 @@ __device__ __forceinline__ float block_max(float v, float* scratch) {
 #define TL_ACT_TANH 8        // tanh(z) (an activation only, never a gate)
 #define TL_ACT_SCALE 9       // a0 z (an activation only, never a gate)
 #define TL_ACT_GELU_TANH 10  // the tanh form: 0.5 x (1 + tanh(sqrt(2 / pi) (x + 0.044715 x^3)))
-#define TL_ACT_GATE_LAST 10  // the last code a gated product's launcher takes
 #define TL_ACT_LAST 10
+
+// The codes a gated product's launcher takes.
+__host__ __device__ __forceinline__ bool tl_is_gate(int act) {
+  return (act >= TL_ACT_SILU && act <= TL_ACT_IDENTITY) || act == TL_ACT_CLAMPED_SWISH || act == TL_ACT_GELU_TANH;
+}
 
 // (1 + tanh(y)) / 2 is the sigmoid of 2 y: what the tanh form of gelu takes it of
 __device__ __forceinline__ float gelu_tanh_argument(float x) { return 1.5957691216057308f * fmaf(0.044715f * x * x, x, x); }

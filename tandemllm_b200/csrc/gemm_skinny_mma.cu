@@ -470,8 +470,8 @@ extern "C" int tl_gemm_skinny_grouped(const void* x, long long ldx, const int* r
                              : (tile_group && tile_row0 && tile_rows && n_tiles)),
              "skinny grouped product: operands must be 16-byte aligned and the plan complete, or at most %d pairs given",
              SKINNY_WARPS * 32);
-  TL_REQUIRE(swiglu >= -TL_ACT_IDENTITY && swiglu <= TL_ACT_GATE_LAST,
-             "skinny grouped product: gate activation %d is not one of 0..%d (or an ungated one, negated)", swiglu, TL_ACT_GATE_LAST);
+  TL_REQUIRE(swiglu <= 0 ? swiglu >= -TL_ACT_IDENTITY : tl_is_gate(swiglu),
+             "skinny grouped product: gate activation %d is none (nor an ungated one, negated)", swiglu);
   TL_REQUIRE(!row_weight || swiglu > 0, "skinny grouped product: row weights need the gated form (activation %d)", swiglu);
   const dim3 grid(ceil_div(N, 16), max_tiles), block(SKINNY_WARPS * 32);
 #define TL_GROUPED(SW_, T_)                                                                                              \

@@ -198,11 +198,11 @@ extern "C" int tl_add_rmsnorm_streams(float* residual, const float* delta, int p
   return launch_add_rmsnorm<NORM_PLAIN>(p, dtype, stream);
 }
 
-// out [rows, inter] = act(gate_up[:, :inter]) * gate_up[:, inter:], act one of TL_ACT_SILU .. TL_ACT_IDENTITY
+// out [rows, inter] = act(gate_up[:, :inter]) * gate_up[:, inter:], act a gate's code (tl_is_gate)
 extern "C" int tl_gated_mul(const void* gate_up, void* out, int rows, int inter, int act, int dtype, cudaStream_t stream) {
   if (rows == 0) return 0;
   TL_REQUIRE(rows > 0 && inter > 0, "gated_mul: rows %d width %d", rows, inter);
-  TL_REQUIRE(act >= TL_ACT_SILU && act <= TL_ACT_GATE_LAST, "gated_mul: gate activation %d is not one of 1..%d", act, TL_ACT_GATE_LAST);
+  TL_REQUIRE(tl_is_gate(act), "gated_mul: gate activation %d is none", act);
   const long long n = (long long)rows * inter;
   const long long most = (long long)sm_count() * 16;
   const int blocks = (int)(ceil_div64(n, 256) < most ? ceil_div64(n, 256) : most);

@@ -702,8 +702,8 @@ extern "C" int tl_gemm_tc(const void* X, long long ldx, long long x_rows, const 
   const bool gated_form = swiglu > 0;
   TL_REQUIRE(!row_weight || (gated_form && tile_group), "tensor-core gemm: row weights need the grouped, gated form (%d)", swiglu);
   TL_REQUIRE(!bias || !swiglu, "tensor-core gemm: a bias with the gated epilogue is not implemented");
-  TL_REQUIRE(swiglu >= -TL_ACT_IDENTITY && swiglu <= TL_ACT_GATE_LAST,
-             "tensor-core gemm: gate activation %d is not one of 0..%d (or an ungated one, negated)", swiglu, TL_ACT_GATE_LAST);
+  TL_REQUIRE(swiglu <= 0 ? swiglu >= -TL_ACT_IDENTITY : tl_is_gate(swiglu),
+             "tensor-core gemm: gate activation %d is none (nor an ungated one, negated)", swiglu);
   TL_REQUIRE(!row_index || (swap && tile_group && row_div >= 1),
              "tensor-core gemm: a row index needs the swapped grouped kernel (divisor %d)", row_div);
   CUtensorMap tmW, tmX;

@@ -309,11 +309,12 @@ def test_silu_mul(dtype):
 def plain_activation(name, g):
     """The gate activations a gated feed-forward may name, in plain torch."""
     return {"silu": torch.nn.functional.silu, "gelu": lambda t: torch.nn.functional.gelu(t),
-            "relu2": lambda t: torch.relu(t) ** 2, "identity": lambda t: t}[name](g)
+            "relu2": lambda t: torch.relu(t) ** 2, "identity": lambda t: t,
+            "gelu_tanh": lambda t: torch.nn.functional.gelu(t, approximate="tanh")}[name](g)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("act", ["silu", "gelu", "relu2", "identity"])
+@pytest.mark.parametrize("act", ["silu", "gelu", "relu2", "identity", "gelu_tanh"])
 def test_gate_activations(dtype, act):
     o = ops()
     gu = rnd(9, 2 * 150, seed=5, scale=1.5).to(dtype)

@@ -661,7 +661,7 @@ def test_pair_product_into_a_wider_output_with_strided_token_rows():
     assert bool(torch.isnan(wide[:, :8]).all()) and bool(torch.isnan(wide[:, 8 + N:]).all())
 
 
-@pytest.mark.parametrize("act", ["silu", "gelu", "relu2", "identity"])
+@pytest.mark.parametrize("act", ["silu", "gelu", "relu2", "identity", "gelu_tanh"])
 @pytest.mark.parametrize("M,H,I", [(300, 136, 200), (40, 64, 72), (1024, 256, 640)])
 def test_pair_product_with_the_gated_epilogue(M, H, I, act):
     from tandemllm_b200.kernels import ops
