@@ -249,7 +249,8 @@ def latent(a) -> dict:
 
 
 def recurrence(a) -> dict:
-    """The recurrence over a matrix state a head of one layer (`--rule delta`, `decay` or `gated`): `batch` requests of `rows` rows."""
+    """The recurrence over a matrix state a head of one layer (`--rule delta`, `decay`, `turned` (a fixed decay, q and k
+    turned by their position) or `gated`): `batch` requests of `rows` rows."""
     from tandemllm_b200.kernels import ops
     ops.core()
     H, D, VD, B, R = a.heads, a.dim, a.vdim, a.batch, a.rows
@@ -267,6 +268,10 @@ def recurrence(a) -> dict:
               rate=0.6, key_eps=1e-6) if delta else dict(head_decay=torch.full((H,), 0.97, device=DEV), silu_inputs=True)
     if a.rule == "gated":       # a decay a key channel and token, sigmoid(w + w0)^rate
         kw = dict(w=torch.randn(B * R, I, device=DEV), w0=torch.full((I,), 3.0, device=DEV), rate=1.0 / 16, q_scale=D ** -0.5)
+    if a.rule == "turned":
+        inv = (1e6 ** (-torch.arange(0, D, 2, dtype=torch.float64) / D)).float().to(DEV)
+        kw = dict(head_decay=torch.full((H,), 0.97, device=DEV), k_scale=D ** -0.5,
+                  turn=(torch.arange(R, dtype=torch.int32, device=DEV).repeat(B) + a.start, inv, D))
     ms = timed(lambda: ops.recurrence_scan(proj, cols["q"], cols["k"], cols["v"], state, slot, start, B, y, H, D, VD,
                                            max_rows=R, **kw), a.iters)
     flops = (10.0 if delta else 6.0) * B * R * H * D * VD
@@ -403,7 +408,8 @@ def main(argv=None) -> int:
     la.add_argument("--kv-rank", type=int, default=256)
     la.add_argument("--rot-dim", type=int, default=32)
     rc = sub.add_parser("recurrence")
-    rc.add_argument("--rule", default="delta", choices=("delta", "decay", "gated", "channel", "head", "memory"))
+    rc.add_argument("--rule", default="delta", choices=("delta", "decay", "turned", "gated", "channel", "head", "memory"))
+    rc.add_argument("--start", type=int, default=1024, help="--rule turned: the position of a request's first row")
     rc.add_argument("--batch", type=int, default=1)
     rc.add_argument("--rows", type=int, default=2048)
     rc.add_argument("--heads", type=int, default=16)

@@ -46,15 +46,20 @@ struct RecTurn {
   float k_scale;
 };
 
-// Entry i (below turn.rot) of q and of k of one head, turned: `q`, `k` its first entries.
-__device__ __forceinline__ void rec_turned(const RecTurn& turn, float pos, const float* __restrict__ q, const float* __restrict__ k,
-                                           int i, float* qv, float* kv) {
-  const int half = turn.rot >> 1, pair = i < half ? i : i - half;
-  float sn, cs;
-  sincosf(pos * turn.inv_freq[pair], &sn, &cs);
-  const float qu = q[pair], qw = q[pair + half], ku = k[pair], kw = k[pair + half];
-  *qv = i < half ? qu * cs - qw * sn : qw * cs + qu * sn;
-  *kv = i < half ? ku * cs - kw * sn : kw * cs + ku * sn;
+// The first turn.rot entries of q and of k of one head (`q`, `k`), turned and multiplied by their factors, to tq and tk: a lane takes
+// both entries of a pair, whose sine and cosine are formed once.
+__device__ __forceinline__ void rec_turn_head(const RecTurn& turn, float pos, const float* __restrict__ q, const float* __restrict__ k,
+                                              float* __restrict__ tq, float* __restrict__ tk, float q_scale, int lane) {
+  const int half = turn.rot >> 1;
+  for (int i = lane; i < half; i += 32) {
+    const float qu = q[i], qw = q[i + half], ku = k[i], kw = k[i + half];
+    float sn, cs;
+    sincosf(pos * turn.inv_freq[i], &sn, &cs);
+    tq[i] = (qu * cs - qw * sn) * q_scale;
+    tq[i + half] = (qw * cs + qu * sn) * q_scale;
+    tk[i] = (ku * cs - kw * sn) * turn.k_scale;
+    tk[i + half] = (kw * cs + ku * sn) * turn.k_scale;
+  }
 }
 
 constexpr int RULE_FIXED = 0, RULE_DELTA = 1, RULE_GATED = 2;
@@ -110,15 +115,13 @@ __global__ void __launch_bounds__(REC_THREADS) recurrence_scan_kernel(
       float* tq = s_q + tw * Dp;
       float* tk = s_k + tw * Dp;
       float ss = 0.f;
-      for (int i = lane; i < Dp; i += 32) {
+      const int plain0 = RULE == RULE_FIXED ? turn.rot : 0;       // entries below have been turned
+      if (plain0 > 0) rec_turn_head(turn, (float)turn.positions[t0 + tw], row + q_col, row + k_col, tq, tk, q_scale, lane);
+      for (int i = plain0 + lane; i < Dp; i += 32) {
         float qv = 0.f, kv = 0.f;
         if (i < D) {
-          if (RULE == RULE_FIXED && i < turn.rot) {
-            rec_turned(turn, (float)turn.positions[t0 + tw], row + q_col, row + k_col, i, &qv, &kv);
-          } else {
-            qv = row[q_col + i];
-            kv = row[k_col + i];
-          }
+          qv = row[q_col + i];
+          kv = row[k_col + i];
           if (silu_inputs) {
             qv = siluf_(qv);
             kv = siluf_(kv);
@@ -249,15 +252,13 @@ __global__ void __launch_bounds__(128) recurrence_prepare_kernel(
   float* tq = prep + ((long long)h * (pairs / H) + r) * NARR * Dp;
   float* tk = tq + Dp;
   float ss = 0.f;
-  for (int i = lane; i < Dp; i += 32) {
+  const int plain0 = RULE == RULE_FIXED ? turn.rot : 0;       // entries below have been turned
+  if (plain0 > 0) rec_turn_head(turn, (float)turn.positions[r], row + q_col, row + k_col, tq, tk, q_scale, lane);
+  for (int i = plain0 + lane; i < Dp; i += 32) {
     float qv = 0.f, kv = 0.f;
     if (i < D) {
-      if (RULE == RULE_FIXED && i < turn.rot) {
-        rec_turned(turn, (float)turn.positions[r], row + q_col, row + k_col, i, &qv, &kv);
-      } else {
-        qv = row[q_col + i];
-        kv = row[k_col + i];
-      }
+      qv = row[q_col + i];
+      kv = row[k_col + i];
       if (silu_inputs) {
         qv = siluf_(qv);
         kv = siluf_(kv);

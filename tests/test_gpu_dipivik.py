@@ -576,3 +576,21 @@ def test_a_model_of_real_layer_widths(dtype):
     toks = {r: torch.randint(0, cfg["vocab"], (n,), generator=g).tolist() for r, n in (("a", 200), ("b", 70))}
     schedule = [[("a", 150)], [("a", 40), ("b", 64)]] + [[("a", 1), ("b", 1)]] * 6 + [[("a", 4)]]
     held_to_the_plain_model(engine, cfg, W, toks, schedule, dtype, "real widths")
+
+
+@pytest.mark.parametrize("only", ["retention", "latent_attention"])
+def test_a_model_of_one_kind_of_layer(only):
+    """Nothing but retention: no page is ever held, only slots. Nothing but latent attention: no state but the last token."""
+    layers = {"retention": [C.retention(2, 16, 8, (100.0, 16), ff=24), C.retention(1, 8, 16, None, ff=None)],
+              "latent_attention": [C.latent(2, 16, 8, 8, 16, 16, 0.2, 100.0, 20, ff=24), C.latent(1, 8, 2, 16, 8, 8, 0.3, 100.0, 20, ff=None)]}
+    from tandemllm_b200.sampling import SamplingParams
+    cfg = C.model(40, 36, 1e-5, layers[only], bigram=(11, 5, 3), cap=8.0)
+    W = C.random_weights(cfg, 3)
+    engine, _, _ = engine_of(None, "float32", cfg=cfg, W=W, pages=12, parallel=2, graph=True, max_len=128, chunk_size=16)
+    g = torch.Generator().manual_seed(1)
+    texts = {r: torch.randint(0, 40, (n,), generator=g).tolist() for r, n in (("a", 60), ("b", 21))}
+    held_to_the_plain_model(engine, cfg, W, texts, [[("a", 33), ("b", 1)], [("a", 2), ("b", 19)], [("b", 1)], [("a", 25)]], "float32", only)
+    outs = engine.generate([texts["a"], texts["b"], texts["a"][:5]], SamplingParams(temperature=0.0, max_tokens=10))
+    for p, o in zip((texts["a"], texts["b"], texts["a"][:5]), outs):
+        assert len(o) == 10
+        agrees_greedily(cfg, W, p, o, "float32")
