@@ -288,6 +288,14 @@ __global__ void __launch_bounds__(192) gemm_tc_kernel(const __grid_constant__ CU
     // ---- epilogue: warp w reads tensor-memory lanes 32 (w % 4) .. + 31 ----
     const int quad = warp & 3;
     const int m_row = quad * 32 + lane;                  // row of the M side this thread owns
+    // (swapped, gated: the weights of the tile's tokens, token lane + 32 i in a lane's i-th, are on their way under the product)
+    constexpr int RW = SWAP && SWIGLU ? (BN + 31) / 32 : 1;
+    float rw[RW];
+    if constexpr (SWAP && SWIGLU) {
+#pragma unroll
+      for (int i = 0; i < RW; ++i)
+        rw[i] = lane + 32 * i < tok_rows ? pair_weight(p.row_weight, p.weight_index, (long long)tok0 + lane + 32 * i) : 1.f;
+    }
     bool ok = num_kb > 0 ? mbar_wait(acc_ready, 0) : true;
     if (num_kb <= 0) chain_wait();      // an empty k range writes zeros, and nothing else has ordered them behind the kernels in front
     if (!ok) {
@@ -308,6 +316,18 @@ __global__ void __launch_bounds__(192) gemm_tc_kernel(const __grid_constant__ CU
 #pragma unroll
           for (int j = 0; j < 16; ++j) v[j] = u[j] = 0.f;
         }
+        if constexpr (SWAP && SWIGLU)
+          if (p.row_weight) {
+            float mine = rw[0];
+#pragma unroll
+            for (int i = 1; i < RW; ++i) mine = (c0 >> 5) == i ? rw[i] : mine;
+#pragma unroll
+            for (int j = 0; j < 16; ++j) {
+              const float wj = __shfl_sync(0xffffffffu, mine, (c0 & 16) + j);
+              v[j] *= wj;
+              u[j] *= wj;
+            }
+          }
         if (SWAP) {
           // this thread: output column n0 + m_row; registers: tokens tok0 + c0 + j
           const int n = n0 + m_row;
@@ -317,8 +337,7 @@ __global__ void __launch_bounds__(192) gemm_tc_kernel(const __grid_constant__ CU
             for (int j = 0; j < 16; ++j) {
               const int t = c0 + j;
               if (t < tok_rows) {
-                const float rw = SWIGLU ? pair_weight(p.row_weight, p.weight_index, tok0 + t) : 1.f;
-                const float r = SWIGLU ? gated(rw * v[j], rw * u[j], p.act, p.ga0, p.ga1) : plain_result(v[j] + b, p.act);
+                const float r = SWIGLU ? gated(v[j], u[j], p.act, p.ga0, p.ga1) : plain_result(v[j] + b, p.act);
                 if (p.partial) p.partial[((long long)blockIdx.z * p.M + tok0 + t) * p.N + n] = r;
                 else store_out<TOut>(C + (long long)(tok0 + t) * p.ldc + n, r);
               }
@@ -328,12 +347,12 @@ __global__ void __launch_bounds__(192) gemm_tc_kernel(const __grid_constant__ CU
           // this thread: token tok0 + m_row; registers: output columns n0 + c0 + j
           if (m_row < tok_rows) {
             TOut* row = C + (long long)(tok0 + m_row) * p.ldc;
-            const float rw = SWIGLU ? pair_weight(p.row_weight, p.weight_index, tok0 + m_row) : 1.f;
+            const float w = SWIGLU ? pair_weight(p.row_weight, p.weight_index, tok0 + m_row) : 1.f;
             float r[16];
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
               const int n = n0 + c0 + j;
-              r[j] = SWIGLU ? gated(rw * v[j], rw * u[j], p.act, p.ga0, p.ga1)
+              r[j] = SWIGLU ? gated(w * v[j], w * u[j], p.act, p.ga0, p.ga1)
                             : plain_result(v[j] + ((p.bias && n < p.N) ? p.bias[n] : 0.f), p.act);
             }
             // 16 consecutive outputs of one row: 16-byte stores when they are all there and aligned

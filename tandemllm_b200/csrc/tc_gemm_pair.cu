@@ -342,6 +342,17 @@ __global__ void __launch_bounds__(Smem<GATED, PER_SM>::THREADS, PER_SM) gemm_tc_
       if (tok_rows <= 0) continue;
       const int n_mma = (tok_rows + 15) & ~15;
       const int buf = n % S::ACC_BUFS, round = n / S::ACC_BUFS;
+      // The weights of the pairs that the warp's blocks of 16 tokens stand for (at most eight blocks: two a register, a block a half of
+      // the lanes) are on their way while the MMAs run.
+      constexpr int STEP = 16 * (S::EPI_WARPS / 4);
+      float rw[4] = {1.f, 1.f, 1.f, 1.f};
+      if (GATED && p.row_weight) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int t = 16 * turn_of + (2 * i + (lane >> 4)) * STEP + (lane & 15);
+          if (t < tok_rows) rw[i] = pair_weight(p.row_weight, p.weight_index, (long long)tok0 + t);
+        }
+      }
       if (num_kb > 0 && !mbar_wait(&acc_full[buf], round & 1)) {
         give_up();
         break;
@@ -356,9 +367,6 @@ __global__ void __launch_bounds__(Smem<GATED, PER_SM>::THREADS, PER_SM) gemm_tc_
 #pragma unroll 1
       for (int c0 = 16 * turn_of; c0 < n_mma; c0 += 16 * (S::EPI_WARPS / 4)) {
         float v[16], u[16];
-        float rw = 1.f;                                              // lane j: the weight of token c0 + j's pair
-        if (GATED && p.row_weight && c0 + (lane & 15) < tok_rows)
-          rw = pair_weight(p.row_weight, p.weight_index, (long long)tok0 + c0 + (lane & 15));
         if (num_kb > 0) {
           ld16(taddr + c0, v);
           if (GATED) ld16(taddr + S::UP_COL + c0, u);
@@ -374,9 +382,11 @@ __global__ void __launch_bounds__(Smem<GATED, PER_SM>::THREADS, PER_SM) gemm_tc_
           // stands outside the 16 independent evaluations, and SiLU, the usual one, takes the fast exponential and
           // division (the result is rounded to bfloat16, far coarser than their error).
           if (p.row_weight) {
+            const int block = c0 / STEP;
+            const float mine = (block >> 1) == 0 ? rw[0] : ((block >> 1) == 1 ? rw[1] : ((block >> 1) == 2 ? rw[2] : rw[3]));
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
-              const float wj = __shfl_sync(0xffffffffu, rw, j);
+              const float wj = __shfl_sync(0xffffffffu, mine, 16 * (block & 1) + j);
               v[j] *= wj;
               u[j] *= wj;
             }
