@@ -132,7 +132,8 @@ __device__ __forceinline__ int nth_set_bit(uint32_t m, int n) {
   return __ffs(m) - 1;
 }
 
-template <bool SWIGLU, typename TOut>
+// WEIGHED: a row's sums are multiplied by its pair's own weight (a kernel of its own, so that the others stay as lean as they are).
+template <bool SWIGLU, bool WEIGHED, typename TOut>
 __global__ void __launch_bounds__(SKINNY_WARPS * 32) gemm_skinny_grouped_kernel(
     const bf16* __restrict__ x, long long ldx, const int* __restrict__ row_index, int row_div, const bf16* __restrict__ w,
     long long ldw, long long rows_per_group, TOut* __restrict__ out, long long ldc, int N, int K,
@@ -145,7 +146,7 @@ __global__ void __launch_bounds__(SKINNY_WARPS * 32) gemm_skinny_grouped_kernel(
   __shared__ float part[SKINNY_WARPS][W_TILES][16][8 + 1];
   __shared__ uint32_t s_match[SKINNY_WARPS];
   __shared__ int s_pair[8];
-  __shared__ float s_weight[8];
+  __shared__ float s_weight[WEIGHED ? 8 : 1];
   chain_next();
   chain_wait();
   const int tile = blockIdx.y;
@@ -223,8 +224,8 @@ __global__ void __launch_bounds__(SKINNY_WARPS * 32) gemm_skinny_grouped_kernel(
   for (int j = 0; j < W_TILES; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
   // (a row's own weight, which the epilogue multiplies its sums by, is on its way under the product)
   float my_weight = 1.f;
-  if constexpr (SWIGLU)
-    if (row_weight && warp == 0 && t == 0 && x_ok) my_weight = pair_weight(row_weight, weight_index, pos);
+  if constexpr (WEIGHED)
+    if (warp == 0 && t == 0 && x_ok) my_weight = pair_weight(row_weight, weight_index, pos);
 
   const int chunks = (K + 31) / 32;
   for (int c0 = warp; c0 < chunks; c0 += SKINNY_WARPS * UNROLL) {
@@ -260,7 +261,7 @@ __global__ void __launch_bounds__(SKINNY_WARPS * 32) gemm_skinny_grouped_kernel(
     part[warp][j][g + 8][2 * t] = acc[j][2];
     part[warp][j][g + 8][2 * t + 1] = acc[j][3];
   }
-  if (SWIGLU && warp == 0 && t == 0) s_weight[g] = my_weight;
+  if (WEIGHED && warp == 0 && t == 0) s_weight[g] = my_weight;
   __syncthreads();
   for (int i = threadIdx.x; i < 16 * 8; i += SKINNY_WARPS * 32) {
     const int row = i & 15, m = i >> 4;
@@ -272,7 +273,11 @@ __global__ void __launch_bounds__(SKINNY_WARPS * 32) gemm_skinny_grouped_kernel(
 #pragma unroll
       for (int s = 0; s < SKINNY_WARPS; ++s) v[j] += part[s][j][row][m];
     }
-    const float r = SWIGLU ? gated(s_weight[m] * v[0], s_weight[m] * v[W_TILES - 1], act, ga0, ga1) : (act < 0 ? gate_activation(v[0], -act) : v[0]);
+    if constexpr (WEIGHED) {
+#pragma unroll
+      for (int j = 0; j < W_TILES; ++j) v[j] *= s_weight[m];
+    }
+    const float r = SWIGLU ? gated(v[0], v[W_TILES - 1], act, ga0, ga1) : (act < 0 ? gate_activation(v[0], -act) : v[0]);
     out[(long long)s_pair[m] * ldc + n0 + row] = from_f32<TOut>(r);
   }
 }
@@ -474,17 +479,21 @@ extern "C" int tl_gemm_skinny_grouped(const void* x, long long ldx, const int* r
              "skinny grouped product: gate activation %d is none (nor an ungated one, negated)", swiglu);
   TL_REQUIRE(!row_weight || swiglu > 0, "skinny grouped product: row weights need the gated form (activation %d)", swiglu);
   const dim3 grid(ceil_div(N, 16), max_tiles), block(SKINNY_WARPS * 32);
-#define TL_GROUPED(SW_, T_)                                                                                              \
-  return (int)launch_chained(gemm_skinny_grouped_kernel<SW_, T_>, grid, block, 0, stream, (const bf16*)x, ldx, row_index,  \
+#define TL_GROUPED(SW_, WE_, T_)                                                                                              \
+  return (int)launch_chained(gemm_skinny_grouped_kernel<SW_, WE_, T_>, grid, block, 0, stream, (const bf16*)x, ldx, row_index,  \
                              row_div, (const bf16*)w, ldw, rows_per_group, (T_*)out, ldc, N, K, tile_group, tile_row0,    \
                              tile_rows, n_tiles, pair_group, n_pairs, n_groups, status, swiglu, tl_gate_constants[0], tl_gate_constants[1],     \
                              row_weight, weight_index, 0u)
   if (swiglu > 0) {
-    if (out_dtype == TL_FP32) TL_GROUPED(true, float);
-    TL_GROUPED(true, bf16);
+    if (row_weight) {
+      if (out_dtype == TL_FP32) TL_GROUPED(true, true, float);
+      TL_GROUPED(true, true, bf16);
+    }
+    if (out_dtype == TL_FP32) TL_GROUPED(true, false, float);
+    TL_GROUPED(true, false, bf16);
   }
-  if (out_dtype == TL_FP32) TL_GROUPED(false, float);
-  TL_GROUPED(false, bf16);
+  if (out_dtype == TL_FP32) TL_GROUPED(false, false, float);
+  TL_GROUPED(false, false, bf16);
 #undef TL_GROUPED
 }
 
